@@ -17,6 +17,8 @@
 // the window; their 16-key units are walked before the window's, by the first split.  `gate`, if given,
 // holds one value per token and query head (row stride `gate_stride`): the head's output is multiplied
 // by its sigmoid where the output is written.
+// `chunk` > 0 (instead of a window): a token sees the keys of its own chunk only.  `cap_out` > 0: scores pass
+// a soft cap, cap * tanh(score / cap), before the softmax.
 // The reference's counterpart is the Triton split-K flash-decoding kernel with the group
 // padded to 16 rows and tiles staged through shared memory (engine/ek_kernels.py:534-615,
 // combine 988-1019; split planning 1355-1381).  Softmax is computed in 32-bit.
@@ -56,7 +58,7 @@ __device__ __forceinline__ uint32_t reg_of(const uint4& v, int i) {
 }
 
 // grid (tokens, kv_heads * row_blocks, splits); DCH = head_dim / 32
-template <int DCH>
+template <int DCH, bool CAP>
 __global__ void __launch_bounds__(kDecWarps * 32)
 attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_stride,
                              const int* positions, const int* token_slot,
@@ -65,7 +67,7 @@ attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_st
                              float* __restrict__ part_acc, float* __restrict__ part_ml,
                              float sink_log2, const float* __restrict__ sinks, int keep_first,
                              const bf16* __restrict__ gate, int gate_stride, int cross,
-                             float* __restrict__ out32) {
+                             float* __restrict__ out32, int chunk, float cap_in, float cap_out) {
   constexpr int D = DCH * 32;
   extern __shared__ float smem[];              // [warps][16][D] accumulators, then [warps][16][2]
   float* o_s = smem;
@@ -89,7 +91,7 @@ attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_st
   int lo = 0, hi = -1;
   int f_hi = -1;                               // kept first keys 0 .. f_hi, before the window
   if (pos >= 0) {
-    lo = window > 0 ? max(0, pos - window + 1) : 0;
+    lo = first_key(pos, window, chunk);
     hi = pos;
     f_hi = min(keep_first, lo) - 1;
     if (n_splits > 1) {
@@ -172,7 +174,8 @@ attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_st
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + 8 * j + 2 * tq + (e & 1);
-          const float v = (key >= m_lo && key <= m_hi) ? s[j][e] * scale_log2 : -INFINITY;
+          const float sc = CAP ? cap_out * tanh_by_exp(s[j][e] * cap_in) : s[j][e] * scale_log2;
+          const float v = (key >= m_lo && key <= m_hi) ? sc : -INFINITY;
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -304,18 +307,19 @@ __global__ void attention_decode_combine_kernel(bf16* __restrict__ out,
   }
 }
 
-template <int DCH>
+template <int DCH, bool CAP = false>
 static int launch_dch(bf16* out, const bf16* q, int q_row_stride, const int* positions,
                       const int* token_slot, PagedKV cache, int n_tokens, int n_q_heads,
                       float scale, int window, int n_splits, int keys_per_split, float* part_acc,
                       float* part_ml, float sink, const float* sinks, int keep_first, const bf16* gate,
-                      int gate_stride, cudaStream_t stream, int cross = 1, float* out32 = nullptr) {
+                      int gate_stride, cudaStream_t stream, int cross = 1, float* out32 = nullptr,
+                      int chunk = 0, float softcap = 0.f) {
   constexpr int D = DCH * 32;
   const int group = n_q_heads / cache.heads;
   const int row_blocks = (group + 15) / 16;
   const size_t smem = (size_t)kDecWarps * 16 * (D + 2) * sizeof(float);
   if (smem > 40 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_bf16_kernel<DCH>,
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_bf16_kernel<DCH, CAP>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
@@ -325,12 +329,13 @@ static int launch_dch(bf16* out, const bf16* q, int q_row_stride, const int* pos
   // stays L1, which the K/V stream needs for its loads in flight
   const int blocks_per_sm = DCH <= 4 ? 3 : 2;
   const int percent = (int)((blocks_per_sm * (smem + 1024) * 100 + 228 * 1024 - 1) / (228 * 1024));
-  prefer_carveout((const void*)attention_decode_bf16_kernel<DCH>, percent < 50 ? 50 : percent);
-  cudaError_t e = launch_pdl(attention_decode_bf16_kernel<DCH>, grid, dim3(kDecWarps * 32), smem,
+  prefer_carveout((const void*)attention_decode_bf16_kernel<DCH, CAP>, percent < 50 ? 50 : percent);
+  cudaError_t e = launch_pdl(attention_decode_bf16_kernel<DCH, CAP>, grid, dim3(kDecWarps * 32), smem,
                              stream, out, q, q_row_stride, positions, token_slot, cache, n_q_heads,
                              row_blocks, scale * 1.4426950408889634f, window, n_splits,
                              keys_per_split, part_acc, part_ml, sink * 1.4426950408889634f, sinks,
-                             window > 0 ? keep_first : 0, gate, gate_stride, cross, out32);
+                             window > 0 ? keep_first : 0, gate, gate_stride, cross, out32, chunk,
+                             CAP ? scale / softcap : 0.f, CAP ? softcap * 1.4426950408889634f : 0.f);
   if (e != cudaSuccess || n_splits == 1) return (int)e;
   dim3 cgrid(n_tokens, n_q_heads * cross);
   return (int)launch_pdl(attention_decode_combine_kernel, cgrid, dim3(64), 0, stream, out,
@@ -351,9 +356,10 @@ EK_EXPORT int ek_attention_decode_bf16(void* out, const void* q, int q_row_strid
                                        int window, int n_splits, int keys_per_split,
                                        float* part_acc, float* part_ml, float sink,
                                        const float* sinks, int keep_first, const void* gate,
-                                       int gate_stride, cudaStream_t stream) {
+                                       int gate_stride, int chunk, float softcap, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
+  if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return EK_ERR_ARG;
   if (head_dim % 32 || head_dim < 32 || head_dim > 256 || n_kv_heads <= 0 ||
       n_q_heads % n_kv_heads || n_splits < 1 || n_splits > 65535 || q_row_stride % 8 ||
       (n_splits > 1 && (!part_acc || !part_ml || keys_per_split < 0 || keys_per_split % kUnit)))
@@ -361,9 +367,15 @@ EK_EXPORT int ek_attention_decode_bf16(void* out, const void* q, int q_row_strid
   PagedKV cache{(void*)k_pages, (void*)v_pages, block_table, table_stride, n_kv_heads, head_dim};
 #define EK_CASE(DCH)                                                                              \
   case DCH:                                                                                       \
+    if (softcap > 0.f)                                                                            \
+      return launch_dch<DCH, true>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot, \
+                                   cache, n_tokens, n_q_heads, scale, window, n_splits, keys_per_split, \
+                                   part_acc, part_ml, sink, sinks, keep_first, (const bf16*)gate, \
+                                   gate_stride, stream, 1, nullptr, chunk, softcap);              \
     return launch_dch<DCH>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot, cache, \
                            n_tokens, n_q_heads, scale, window, n_splits, keys_per_split, part_acc, \
-                           part_ml, sink, sinks, keep_first, (const bf16*)gate, gate_stride, stream);
+                           part_ml, sink, sinks, keep_first, (const bf16*)gate, gate_stride, stream, 1,   \
+                           nullptr, chunk, softcap);
   switch (head_dim / 32) {
     EK_CASE(1) EK_CASE(2) EK_CASE(3) EK_CASE(4) EK_CASE(5) EK_CASE(6) EK_CASE(7) EK_CASE(8)
   }
@@ -465,5 +477,5 @@ EK_EXPORT int ek_attention_decode_bf16_noalloc(void* out, const void* q, int q_r
   return ek_attention_decode_bf16(out, q, q_row_stride, positions, token_slot, k_pages, v_pages,
                                   block_table, table_stride, n_tokens, n_q_heads, n_kv_heads,
                                   head_dim, scale, window, n_splits, keys_per_split, part_acc,
-                                  part_ml, -INFINITY, nullptr, 0, nullptr, 0, stream);
+                                  part_ml, -INFINITY, nullptr, 0, nullptr, 0, 0, 0.f, stream);
 }

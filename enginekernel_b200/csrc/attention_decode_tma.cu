@@ -69,7 +69,8 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
                             const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
-                            int window, int* status, float sink_log2) {
+                            int window, int* status, float sink_log2, int chunk, float cap_in,
+                            float cap_out) {
   constexpr int DB = D / 64;                       // 64-wide (128-byte) blocks of the head dimension
   constexpr uint32_t kSub = EK_PAGE * 128;         // one [64 keys x 64 dims] sub-tile: 8 KB
   constexpr uint32_t kStage = 2 * DB * kSub;       // K tile + V tile
@@ -107,7 +108,7 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
   const int pos = positions[t];
   int lo = 0, hi = -1, pg_first = 0, pg_last = -1;
   if (pos >= 0) {
-    lo = window > 0 ? max(0, pos - window + 1) : 0;
+    lo = first_key(pos, window, chunk);
     hi = pos;
     const int pg_lo = lo / EK_PAGE, pg_hi = hi / EK_PAGE;
     const int per = (pg_hi - pg_lo + n_splits) / n_splits;     // pages a split, rounded up
@@ -204,7 +205,8 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int key = key0 + 8 * j + 2 * tq + (e & 1);
-              const float v = (key >= lo && key <= hi) ? sc[j][e] * scale_log2 : -INFINITY;
+              const float score = cap_out > 0.f ? cap_out * tanh_by_exp(sc[j][e] * cap_in) : sc[j][e] * scale_log2;
+              const float v = (key >= lo && key <= hi) ? score : -INFINITY;
               sc[j][e] = v;
               mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
@@ -351,7 +353,7 @@ static int launch_dt(bf16* out, const bf16* q, int q_row_stride, const int* posi
                      const int* token_slot, const void* k_pages, const void* v_pages,
                      long long page_rows, const int* block_table, int table_stride, int n_tokens,
                      int n_q_heads, int n_kv_heads, float scale, int window, int n_splits, int* status,
-                     float sink, cudaStream_t stream) {
+                     float sink, int chunk, float softcap, cudaStream_t stream) {
   constexpr int STAGES = (D == 128 ? 3 : 6) * (DEEP ? 2 : 1);
   constexpr int DB = D / 64;
   constexpr size_t smem = 1024 + (size_t)STAGES * 2 * DB * EK_PAGE * 128 + 2 * STAGES * 8 +
@@ -401,11 +403,12 @@ static int launch_dt(bf16* out, const bf16* q, int q_row_stride, const int* posi
                                      q_row_stride, positions, token_slot, mk, mv, block_table,
                                      table_stride, n_kv_heads, n_q_heads,
                                      scale * 1.4426950408889634f, window, status,
-                         sink * 1.4426950408889634f);
+                                     sink * 1.4426950408889634f, chunk, softcap > 0.f ? scale / softcap : 0.f,
+                                     softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
   return (int)launch_pdl(kernel, grid, dim3(kDtThreads), smem, stream, out, q, q_row_stride, positions,
                          token_slot, mk, mv, block_table, table_stride, n_kv_heads, n_q_heads,
-                         scale * 1.4426950408889634f, window, status,
-                         sink * 1.4426950408889634f);
+                         scale * 1.4426950408889634f, window, status, sink * 1.4426950408889634f, chunk,
+                         softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
 }
 
 }  // namespace ek
@@ -417,10 +420,10 @@ EK_EXPORT int ek_attention_decode_tma_max_splits(int head_dim) {
   int clusters = 0;
   if (head_dim == 64)
     clusters = launch_dt<64, false, true>(nullptr, nullptr, 0, nullptr, nullptr, &clusters, &clusters, 64,
-                                          nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, nullptr);
+                                          nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, 0, 0.f, nullptr);
   else if (head_dim == 128)
     clusters = launch_dt<128, false, true>(nullptr, nullptr, 0, nullptr, nullptr, &clusters, &clusters, 64,
-                                           nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, nullptr);
+                                           nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, 0, 0.f, nullptr);
   else
     return 0;
   return clusters >= 1 ? kDtMaxSplits : kDtPortableSplits;
@@ -430,16 +433,18 @@ EK_EXPORT int ek_attention_decode_tma_max_splits(int head_dim) {
 // the token's visible range); q rows 4-byte aligned; n_pages = pages in k_pages / v_pages
 // ([pages, kv heads, 64, head_dim]); `status` is one int on the device.  `sink`: score of a key
 // without a value that every query also sees (one more term in the softmax denominator);
-// -INFINITY for none.
+// -INFINITY for none.  `chunk` > 0 instead of a window: keys of the token's own chunk of positions only.
+// `softcap` > 0: scores become softcap tanh(score / softcap).
 EK_EXPORT int ek_attention_decode_tma(void* out, const void* q, int q_row_stride,
                                       const int* positions, const int* token_slot,
                                       const void* k_pages, const void* v_pages, int n_pages,
                                       const int* block_table, int table_stride, int n_tokens,
                                       int n_q_heads, int n_kv_heads, int head_dim, float scale,
-                                      int window, int n_splits, int* status, float sink,
-                                      cudaStream_t stream) {
+                                      int window, int n_splits, int* status, float sink, int chunk,
+                                      float softcap, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
+  if (chunk < 0 || (chunk > 0 && window > 0)) return EK_ERR_ARG;
   if ((head_dim != 64 && head_dim != 128) || n_kv_heads <= 0 || n_q_heads % n_kv_heads ||
       n_q_heads / n_kv_heads > 16 || n_splits < 1 || n_splits > kDtMaxSplits || q_row_stride % 2 ||
       ((uintptr_t)q & 3) || !status || n_kv_heads > 65535 || n_tokens > 65535 || n_pages <= 0)
@@ -450,7 +455,8 @@ EK_EXPORT int ek_attention_decode_tma(void* out, const void* q, int q_row_stride
 #define EK_DT(D_, DEEP_)                                                                          \
   return launch_dt<D_, DEEP_>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot,     \
                               k_pages, v_pages, page_rows, block_table, table_stride, n_tokens,   \
-                              n_q_heads, n_kv_heads, scale, window, n_splits, status, sink, stream)
+                              n_q_heads, n_kv_heads, scale, window, n_splits, status, sink, chunk,     \
+                              softcap, stream)
   if (head_dim == 64) {
     if (deep) EK_DT(64, true);
     EK_DT(64, false);

@@ -12,6 +12,8 @@
 // `cross` > 1 (entry point ..._cross): every head's weights are applied to the values of every key/value
 // head and the results are kept in 32-bit, for designs that mix the heads' weights behind the softmax;
 // mix_heads_kernel forms the mixed results from them.
+// `chunk` > 0 (instead of a window): a token sees the keys of its own chunk only, chunks being counted from
+// the sequence's first position.  `softcap` > 0: a score s becomes softcap * tanh(s / softcap) before the softmax.
 // It serves whole prompts, chunks and single decoded tokens alike, since each token
 // carries its own position and slot; the faster bfloat16 kernels in attention_bf16.cu
 // cover the common head sizes, this one covers everything and is the 32-bit path.
@@ -77,7 +79,7 @@ __global__ void attention_generic_kernel(T* __restrict__ out, const T* __restric
                                          float* __restrict__ part_ml, float sink,
                                          const float* __restrict__ sinks, int keep_first,
                                          const T* __restrict__ gate, int gate_stride, int cross,
-                                         float* __restrict__ out32) {
+                                         float* __restrict__ out32, int chunk, float softcap) {
   __shared__ float q_s[kGenericMaxDim];
   __shared__ float p_s[kAttnThreads];
   __shared__ size_t voff_s[kAttnThreads];
@@ -97,7 +99,7 @@ __global__ void attention_generic_kernel(T* __restrict__ out, const T* __restric
   int lo = 0, hi = -1;                          // keys [lo, hi] ...
   int f_lo = 0, f_hi = -1;                      // ... and the kept first keys [f_lo, f_hi] before them
   if (pos >= 0) {
-    lo = window > 0 ? max(0, pos - window + 1) : 0;
+    lo = first_key(pos, window, chunk);
     hi = pos;
     f_hi = min(keep_first, lo) - 1;
     if (n_splits > 1) {
@@ -131,6 +133,7 @@ __global__ void attention_generic_kernel(T* __restrict__ out, const T* __restric
         const int page = table[j / EK_PAGE];
         voff_s[tid] = page_offset(cache, page, v_head, j);
         s = dot_row<T>(kbase + page_offset(cache, page, kv_head, j), q_s, d);
+        if (softcap > 0.f) s = softcap * tanhf(s / softcap);
       }
       const float m_new = fmaxf(m, block_max(s, scratch));
       const float p = seen ? expf(s - m_new) : 0.f;
@@ -211,9 +214,10 @@ static int launch(void* out, const void* q, int q_row_stride, const int* positio
                   int n_kv_heads, int head_dim, float scale, int window, int n_splits,
                   int keys_per_split, float* part_acc, float* part_ml, float sink,
                   const float* sinks, int keep_first, const void* gate, int gate_stride,
-                  cudaStream_t stream, int cross = 1, float* out32 = nullptr) {
+                  cudaStream_t stream, int cross = 1, float* out32 = nullptr, int chunk = 0,
+                  float softcap = 0.f) {
   if (n_tokens <= 0) return 0;
-  if (head_dim <= 0 || head_dim > kGenericMaxDim || n_kv_heads <= 0 ||
+  if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0)) || head_dim <= 0 || head_dim > kGenericMaxDim || n_kv_heads <= 0 ||
       n_q_heads % n_kv_heads || n_q_heads > 65535 || n_splits < 1 || n_splits > 65535 ||
       (n_splits > 1 && (!part_acc || !part_ml || keys_per_split <= 0)) ||
       (cross != 1 && cross != n_kv_heads) || (long long)n_q_heads * cross > 65535)
@@ -223,7 +227,7 @@ static int launch(void* out, const void* q, int q_row_stride, const int* positio
   attention_generic_kernel<T><<<grid, kAttnThreads, 0, stream>>>(
       (T*)out, (const T*)q, q_row_stride, positions, token_slot, cache, n_q_heads, scale, window,
       n_splits, keys_per_split, part_acc, part_ml, sink, sinks, window > 0 ? keep_first : 0,
-      (const T*)gate, gate_stride, cross, out32);
+      (const T*)gate, gate_stride, cross, out32, chunk, softcap);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess || n_splits == 1) return (int)e;
   dim3 cgrid(n_tokens, n_q_heads * cross);
@@ -281,12 +285,12 @@ __global__ void mix_heads_kernel(T* __restrict__ out, const float* __restrict__ 
       const void* k_pages, const void* v_pages, const int* block_table, int table_stride,      \
       int n_tokens, int n_q_heads, int n_kv_heads, int head_dim, float scale, int window,      \
       int n_splits, int keys_per_split, float* part_acc, float* part_ml, float sink,           \
-      const float* sinks, int keep_first, const void* gate, int gate_stride,                   \
-      cudaStream_t stream) {                                                                   \
+      const float* sinks, int keep_first, const void* gate, int gate_stride, int chunk,        \
+      float softcap, cudaStream_t stream) {                                                                \
     return ek::launch<T>(out, q, q_row_stride, positions, token_slot, k_pages, v_pages,        \
                          block_table, table_stride, n_tokens, n_q_heads, n_kv_heads, head_dim, \
                          scale, window, n_splits, keys_per_split, part_acc, part_ml, sink,     \
-                         sinks, keep_first, gate, gate_stride, stream);                        \
+                         sinks, keep_first, gate, gate_stride, stream, 1, nullptr, chunk, softcap); \
   }
 
 #define EK_INSTANTIATE_CROSS(SUFFIX, T)                                                        \

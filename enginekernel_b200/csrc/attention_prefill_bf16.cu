@@ -14,6 +14,8 @@
 // later row, beside its window - the tiles that hold them are walked before the window's.  `gate`, if
 // given, holds one value per token and query head (row stride `gate_stride`): the head's output is
 // multiplied by its sigmoid.
+// `chunk` > 0 (instead of a window): a row sees the keys of its own chunk only, chunks being counted from the
+// sequence's first position.  `cap_out` > 0: scores pass a soft cap, cap * tanh(score / cap), before the softmax.
 // Tiles are found from cu_seqlens on the device (no host-built schedule).
 // The reference's counterpart is a Triton kernel over a padded rectangle, 128x128 tiles,
 // probabilities rounded to bfloat16 before P.V as here (engine/ek_kernels.py:166-221),
@@ -65,7 +67,7 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
                               int n_q_heads, float scale_log2, int window, int tok_per_tile,
                               float sink_log2, const float* __restrict__ sinks, int keep_first,
                               const bf16* __restrict__ gate, int gate_stride, int cross,
-                              float* __restrict__ out32) {
+                              float* __restrict__ out32, int chunk, float cap_in, float cap_out) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int tile_info[3];                 // first token (packed index), tokens, sequence
   const int D = cache.head_dim;
@@ -115,7 +117,7 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
   const int slot = token_slot[t_first];
   const int* table = cache.block_table + (size_t)slot * cache.table_stride;
   const int hi_tile = pos0 + n_tok - 1;
-  const int lo_tile = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int lo_tile = first_key(pos0, window, chunk);
   const int kt_lo = lo_tile / kPfKeys, kt_hi = hi_tile / kPfKeys;
   // tiles of kept first keys that the window's tiles do not cover: 0 .. n_first - 1
   const int n_first = keep_first > 0 ? min((keep_first + kPfKeys - 1) / kPfKeys, kt_lo) : 0;
@@ -162,6 +164,10 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
   const int warp_pos_min = pos0 + (warp * 16) / group;
   const int warp_pos_max = pos0 + min((warp * 16 + 15) / group, n_tok - 1);
   const bool warp_active = warp * 16 < n_rows;
+  // the first key each of them sees, and the lowest and highest of these in the warp
+  const int first_lo = first_key(pos_lo, window, chunk), first_hi = first_key(pos_hi, window, chunk);
+  const int warp_first_min = first_key(warp_pos_min, window, chunk);
+  const int warp_first_max = first_key(warp_pos_max, window, chunk);
 
   for (int it = 0; it < n_tiles; ++it) {
     const int kt = tile_of(it);
@@ -174,7 +180,7 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
     const int key0 = kt * kPfKeys;
     // a warp skips tiles none of its rows can see
     const bool tile_visible = warp_active && key0 <= warp_pos_max &&
-                              (window <= 0 || key0 + kPfKeys - 1 > warp_pos_min - window || key0 < keep_first);
+                              (key0 + kPfKeys - 1 >= warp_first_min || key0 < keep_first);
     if (tile_visible) {
       const bf16* kb = k_s + buf * kPfKeys * LD;
       const bf16* vb = v_s + buf * kPfKeys * LD;
@@ -198,18 +204,17 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
         }
       }
       // scale and mask.  s[j][e]: row (e < 2 ? lo : hi), key key0 + 8j + 2tq + (e & 1)
-      const bool need_mask = key0 + kPfKeys - 1 > warp_pos_min ||
-                             (window > 0 && key0 <= warp_pos_max - window);
+      const bool need_mask = key0 + kPfKeys - 1 > warp_pos_min || key0 < warp_first_max;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int j = 0; j < kPfKeys / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          float v = s[j][e] * scale_log2;
+          float v = cap_out > 0.f ? cap_out * tanh_by_exp(s[j][e] * cap_in) : s[j][e] * scale_log2;
           if (need_mask) {
             const int key = key0 + 8 * j + 2 * tq + (e & 1);
             const int p = e < 2 ? pos_lo : pos_hi;
-            if (key > p || (window > 0 && key <= p - window && key >= keep_first)) v = -INFINITY;
+            if (key > p || (key < (e < 2 ? first_lo : first_hi) && key >= keep_first)) v = -INFINITY;
           }
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -324,7 +329,8 @@ static int launch_dmax(bf16* out, const bf16* q, int q_row_stride, const int* po
                        const int* token_slot, const int* cu_seqlens, int n_seqs, int n_tokens,
                        PagedKV cache, int n_q_heads, float scale, int window, float sink,
                        const float* sinks, int keep_first, const bf16* gate, int gate_stride,
-                       cudaStream_t stream, int cross = 1, float* out32 = nullptr) {
+                       cudaStream_t stream, int cross = 1, float* out32 = nullptr, int chunk = 0,
+                       float softcap = 0.f) {
   const int group = n_q_heads / cache.heads;
   const int tok_per_tile = kPfRows / group;
   const int D = cache.head_dim, LD = D + 8;
@@ -339,7 +345,8 @@ static int launch_dmax(bf16* out, const bf16* q, int q_row_stride, const int* po
   attention_prefill_bf16_kernel<DMAX><<<grid, kPfWarps * 32, smem, stream>>>(
       out, q, q_row_stride, positions, token_slot, cu_seqlens, n_seqs, cache, n_q_heads,
       scale * 1.4426950408889634f, window, tok_per_tile, sink * 1.4426950408889634f, sinks,
-      window > 0 ? keep_first : 0, gate, gate_stride, cross, out32);
+      window > 0 ? keep_first : 0, gate, gate_stride, cross, out32, chunk,
+      softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -382,9 +389,11 @@ EK_EXPORT int ek_attention_prefill_bf16(void* out, const void* q, int q_row_stri
                                         const int* block_table, int table_stride, int n_q_heads,
                                         int n_kv_heads, int head_dim, float scale, int window,
                                         float sink, const float* sinks, int keep_first,
-                                        const void* gate, int gate_stride, cudaStream_t stream) {
+                                        const void* gate, int gate_stride, int chunk, float softcap,
+                                        cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
+  if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return EK_ERR_ARG;
   if (head_dim % 16 || head_dim < 16 || head_dim > 256 || n_kv_heads <= 0 ||
       n_q_heads % n_kv_heads || n_q_heads / n_kv_heads > kPfRows || q_row_stride % 8)
     return EK_ERR_ARG;
@@ -392,12 +401,12 @@ EK_EXPORT int ek_attention_prefill_bf16(void* out, const void* q, int q_row_stri
   if (head_dim <= 64)
     return launch_dmax<64>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot,
                            cu_seqlens, n_seqs, n_tokens, cache, n_q_heads, scale, window, sink, sinks,
-                           keep_first, (const bf16*)gate, gate_stride, stream);
+                           keep_first, (const bf16*)gate, gate_stride, stream, 1, nullptr, chunk, softcap);
   if (head_dim <= 128)
     return launch_dmax<128>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot,
                             cu_seqlens, n_seqs, n_tokens, cache, n_q_heads, scale, window, sink, sinks,
-                           keep_first, (const bf16*)gate, gate_stride, stream);
+                           keep_first, (const bf16*)gate, gate_stride, stream, 1, nullptr, chunk, softcap);
   return launch_dmax<256>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot,
                           cu_seqlens, n_seqs, n_tokens, cache, n_q_heads, scale, window, sink, sinks,
-                           keep_first, (const bf16*)gate, gate_stride, stream);
+                           keep_first, (const bf16*)gate, gate_stride, stream, 1, nullptr, chunk, softcap);
 }

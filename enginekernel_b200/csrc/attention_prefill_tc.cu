@@ -67,14 +67,18 @@ __device__ __forceinline__ float2 add2(float2 a, float2 b) {
   return d;
 }
 
-template <int D>
+// CAP: scores pass a soft cap before the softmax, cap tanh(score / cap): `cap_in` is scale / cap and
+// `scale_log2` then stands for cap log2(e), which multiplies the tanh.  `chunk` > 0 (instead of a window): a
+// row sees the keys of its own chunk of positions only.
+template <int D, bool CAP>
 __global__ void __launch_bounds__(kFaThreads, 2)
 attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUtensorMap map_q,
                             const int4* __restrict__ tiles,
                             const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
-                            int window, int tok_per_tile, int* status, float sink_log2) {
+                            int window, int tok_per_tile, int* status, float sink_log2, int chunk,
+                            float cap_in) {
   constexpr int DB = D / 64;                       // 64-wide blocks of the head dimension
   constexpr uint32_t kSub = kFaKeys * 128;         // one [64 x 64] bfloat16 sub-tile: 8 KB
   constexpr uint32_t kTmemCols = 256;
@@ -136,7 +140,7 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
   }
   const int* table = block_table + (size_t)tile.w * table_stride;
   const int hi_tile = pos0 + n_tok - 1;
-  const int lo_tile = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int lo_tile = first_key(pos0, window, chunk);
   const int kt_lo = lo_tile / kFaKeys, kt_hi = hi_tile / kFaKeys;
   const int n_iter = kt_hi - kt_lo + 1;
   pdl_wait();                                      // Q and the newest keys and values: the kernel ahead
@@ -223,6 +227,7 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
   const uint32_t lane_addr = tmem_base + ((uint32_t)((warp & 3) * 32) << 16);
   if (tid < kFaRows) {
     const int pos_r = pos0 + min(r / group, n_tok - 1);
+    const int first_r = first_key(pos_r, window, chunk);   // the first key this row sees
     for (int it = 0; it < n_iter && ok; ++it) {
       const int s = it & 1;
       const uint32_t phase = (it >> 1) & 1;
@@ -234,7 +239,7 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
       // two blocks of 7 warps an SM set: first the maximum (keys 32..63 are only looked at,
       // keys 0..31 stay in registers), then the exponentials of keys 0..31, their P, and the
       // same for keys 32..63, read from TMEM once more.
-      const bool full = key0 + kFaKeys - 1 <= pos_r && (window <= 0 || key0 > pos_r - window);
+      const bool full = key0 + kFaKeys - 1 <= pos_r && key0 >= first_r;
       auto load_half = [&](int h, float* v) {      // scores of keys key0 + 32 h .., masked
         tmem_ld32_nowait(lane_addr + kColS + 64 * s + 32 * h, v);
         tmem_ld_wait();
@@ -242,7 +247,7 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int key = key0 + 32 * h + i;
-            const bool seen = key <= pos_r && (window <= 0 || key > pos_r - window);
+            const bool seen = key <= pos_r && key >= first_r;
             v[i] = seen ? v[i] : -INFINITY;
           }
         }
@@ -255,7 +260,9 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
       load_half(0, sc);
 #pragma unroll
       for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sc[i]);
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+      float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+      if (CAP && mx > -INFINITY) mx = tanh_by_exp(mx * cap_in);   // (monotonic: the maximum's cap is the caps' maximum)
+      mx *= scale_log2;
       // tcgen05.ld/st are warp-wide: if any row of the warp raises its reference, the whole warp
       // rescales (rows that keep theirs multiply by 1)
       const bool raise = mx > m_ref + kLazy;       // also the first page with a visible key
@@ -291,6 +298,10 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
         uint32_t w[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
+          if (CAP) {                               // (a masked score stays what it is)
+            sc[i] = sc[i] > -INFINITY ? tanh_by_exp(sc[i] * cap_in) : sc[i];
+            sc[i + 1] = sc[i + 1] > -INFINITY ? tanh_by_exp(sc[i + 1] * cap_in) : sc[i + 1];
+          }
           const float2 a = fma2(make_float2(sc[i], sc[i + 1]), scale2, shift2);
           const float2 p = make_float2(ex2_approx(a.x), ex2_approx(a.y));
           psum[(i >> 1) & 1] = add2(psum[(i >> 1) & 1], p);
@@ -441,11 +452,12 @@ attention_prefill_tiles_kernel(int4* tiles, int max_tiles, const int* cu_seqlens
   for (int i = total + tid; i < max_tiles; i += kFaTileThreads) tiles[i] = make_int4(0, 0, -1, 0);
 }
 
-template <int D>
+template <int D, bool CAP>
 static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* tiles, int n_tiles, int n_tokens,
                      const void* k_pages, const void* v_pages, long long page_rows,
                      const int* block_table, int table_stride, int n_q_heads, int n_kv_heads,
-                     float scale, int window, int* status, float sink, cudaStream_t stream) {
+                     float scale, int window, int* status, float sink, int chunk, float softcap,
+                     cudaStream_t stream) {
   const int group = n_q_heads / n_kv_heads;
   const int tok_per_tile = kFaRows / group;
   CUtensorMap mq, mk, mv;
@@ -455,7 +467,7 @@ static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* til
   if ((rc = tensor_map(v_pages, page_rows, D, D, kFaKeys, &mv))) return rc;
   constexpr int DB = D / 64;
   constexpr size_t smem = (size_t)(2 * DB + (kFaKStages + kFaVStages) * DB) * kFaKeys * 128 + kFaBars * 8 + 16;
-  auto kernel = attention_prefill_tc_kernel<D>;
+  auto kernel = attention_prefill_tc_kernel<D, CAP>;
   static bool configured[kMaxDevices] = {};
   int device = 0;
   cudaError_t e = cudaGetDevice(&device);
@@ -470,8 +482,9 @@ static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* til
   if (n_tiles > 65535) return EK_ERR_ARG;
   dim3 grid(n_kv_heads, n_tiles);
   return (int)launch_pdl(kernel, grid, dim3(kFaThreads), smem, stream, out, mq, tiles, mk, mv, block_table,
-                         table_stride, n_kv_heads, n_q_heads, scale * 1.4426950408889634f, window,
-                         tok_per_tile, status, sink * 1.4426950408889634f);
+                         table_stride, n_kv_heads, n_q_heads, (CAP ? softcap : scale) * 1.4426950408889634f,
+                         window, tok_per_tile, status, sink * 1.4426950408889634f, chunk,
+                         CAP ? scale / softcap : 0.f);
 }
 
 }  // namespace ek
@@ -495,25 +508,32 @@ EK_EXPORT int ek_attention_prefill_tiles(int* tiles, int max_tiles, const int* c
 // aligned; n_pages = number of pages in k_pages / v_pages ([pages, kv heads, 64, head_dim]);
 // `tiles` / n_tiles: the table ek_attention_prefill_tiles made for this step and group size.
 // `sink`: score of a key without a value that every query also sees (one more term in the softmax
-// denominator); -INFINITY for none.
+// denominator); -INFINITY for none.  `chunk` > 0 instead of a window: keys of a token's own chunk only.
+// `softcap` > 0: scores become softcap tanh(score / softcap).
 EK_EXPORT int ek_attention_prefill_tc(void* out, const void* q, int q_row_stride, const int* tiles,
                                       int n_tiles, int n_tokens,
                                       const void* k_pages, const void* v_pages, int n_pages,
                                       const int* block_table, int table_stride, int n_q_heads,
                                       int n_kv_heads, int head_dim, float scale, int window,
-                                      int* status, float sink, cudaStream_t stream) {
+                                      int* status, float sink, int chunk, float softcap,
+                                      cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0 || n_tiles <= 0) return 0;
+  if (chunk < 0 || (chunk > 0 && window > 0)) return EK_ERR_ARG;
   if ((head_dim != 64 && head_dim != 128) || n_kv_heads <= 0 || n_q_heads % n_kv_heads ||
       kFaRows % (n_q_heads / n_kv_heads) || q_row_stride % 8 || ((uintptr_t)q & 15) || !status ||
       !(scale > 0.f) || n_pages <= 0 || !tiles || ((uintptr_t)tiles & 15))
     return EK_ERR_ARG;
   const long long page_rows = (long long)n_pages * n_kv_heads * EK_PAGE;
-  if (head_dim == 64)
-    return launch_fa<64>((bf16*)out, (const bf16*)q, q_row_stride, (const int4*)tiles, n_tiles, n_tokens,
-                         k_pages, v_pages, page_rows, block_table, table_stride,
-                         n_q_heads, n_kv_heads, scale, window, status, sink, stream);
-  return launch_fa<128>((bf16*)out, (const bf16*)q, q_row_stride, (const int4*)tiles, n_tiles, n_tokens,
-                        k_pages, v_pages, page_rows, block_table, table_stride,
-                        n_q_heads, n_kv_heads, scale, window, status, sink, stream);
+#define EK_FA(D_, CAP_)                                                                                  \
+  return launch_fa<D_, CAP_>((bf16*)out, (const bf16*)q, q_row_stride, (const int4*)tiles, n_tiles,       \
+                             n_tokens, k_pages, v_pages, page_rows, block_table, table_stride, n_q_heads, \
+                             n_kv_heads, scale, window, status, sink, chunk, softcap, stream)
+  if (head_dim == 64) {
+    if (softcap > 0.f) EK_FA(64, true);
+    EK_FA(64, false);
+  }
+  if (softcap > 0.f) EK_FA(128, true);
+  EK_FA(128, false);
+#undef EK_FA
 }

@@ -113,6 +113,17 @@ __device__ __forceinline__ size_t page_offset(const PagedKV& c, int page, int he
   return (((size_t)page * c.heads + head) * EK_PAGE + (pos & (EK_PAGE - 1))) * (size_t)c.head_dim;
 }
 
+// The first position a token at `pos` sees: the start of its own chunk (chunks of `chunk` positions counted
+// from the sequence's first token), or of its sliding window, or the sequence's start.
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  if (chunk > 0) return pos - pos % chunk;
+  return window > 0 ? max(0, pos - window + 1) : 0;
+}
+
+// tanh for the soft cap of attention scores in the 16-bit kernels: 1 - 2 / (e^(2x) + 1), whose absolute error
+// is a few 32-bit roundings of 1 (the exponential overflows to infinity and the quotient to 0 for large x).
+__device__ __forceinline__ float tanh_by_exp(float x) { return 1.f - __fdividef(2.f, __expf(fminf(2.f * x, 80.f)) + 1.f); }
+
 // Programmatic dependent launch: a kernel launched with `launch_pdl` may start while the
 // kernel before it on the stream is still draining.  It must call `pdl_wait()` before it
 // reads anything that kernel wrote or writes anything that kernel reads (only constants -

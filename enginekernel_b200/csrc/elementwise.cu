@@ -397,8 +397,21 @@ __global__ void bias_act_kernel(T* __restrict__ out, const void* __restrict__ x,
   out[i] = from_f<T>(v);
 }
 
+// ACT 0, 1: silu_of(g) * u.  ACT 2, a gate whose halves are clamped: with g' = min(g, limit) and u' = clamp(u,
+// -limit, limit), g' sigmoid(1.702 g') (u' + 1).
+template <typename T, int ACT>
+__device__ __forceinline__ float gated_of(float g, float u, float limit) {
+  if (ACT == 2) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.f;
+    if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-1.702f * g)) * u;
+    return g / (1.f + expf(-1.702f * g)) * u;
+  }
+  return silu_of<T, ACT>(g) * u;
+}
+
 template <typename T, bool VEC, int ACT>
-__global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, int inter) {
+__global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, int inter, float limit) {
   const size_t r = blockIdx.y;
   const T* g_row = gu + r * 2 * inter;
   T* o_row = out + r * inter;
@@ -406,19 +419,19 @@ __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, i
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
     if (i >= inter) return;
     const float4 g = Vec4<T>::load(g_row + i), u = Vec4<T>::load(g_row + inter + i);
-    Vec4<T>::store(o_row + i, make_float4(silu_of<T, ACT>(g.x) * u.x, silu_of<T, ACT>(g.y) * u.y,
-                                          silu_of<T, ACT>(g.z) * u.z, silu_of<T, ACT>(g.w) * u.w));
+    Vec4<T>::store(o_row + i, make_float4(gated_of<T, ACT>(g.x, u.x, limit), gated_of<T, ACT>(g.y, u.y, limit),
+                                          gated_of<T, ACT>(g.z, u.z, limit), gated_of<T, ACT>(g.w, u.w, limit)));
   } else {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= inter) return;
     const float g = to_f<T>(g_row[i]), u = to_f<T>(g_row[inter + i]);
-    o_row[i] = from_f<T>(silu_of<T, ACT>(g) * u);
+    o_row[i] = from_f<T>(gated_of<T, ACT>(g, u, limit));
   }
 }
 
 // The same for bfloat16 rows whose halves start on 16-byte boundaries: eight neighbours a thread.
 template <int ACT>
-__global__ void silu_mul_wide_kernel(bf16* __restrict__ out, const bf16* __restrict__ gu, int inter) {
+__global__ void silu_mul_wide_kernel(bf16* __restrict__ out, const bf16* __restrict__ gu, int inter, float limit) {
   const size_t r = blockIdx.y;
   const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
   if (i >= inter) return;
@@ -431,7 +444,7 @@ __global__ void silu_mul_wide_kernel(bf16* __restrict__ out, const bf16* __restr
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     const float2 a = __bfloat1622float2(g2[j]), b = __bfloat1622float2(u2[j]);
-    __nv_bfloat162 h = __floats2bfloat162_rn(silu_of<bf16, ACT>(a.x) * b.x, silu_of<bf16, ACT>(a.y) * b.y);
+    __nv_bfloat162 h = __floats2bfloat162_rn(gated_of<bf16, ACT>(a.x, b.x, limit), gated_of<bf16, ACT>(a.y, b.y, limit));
     w[j] = *reinterpret_cast<uint32_t*>(&h);
   }
   *reinterpret_cast<uint4*>(out + r * inter + i) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -466,19 +479,19 @@ static int launch_rmsnorm(void* y, float* resid, const void* add, const float* g
 }
 
 template <typename T, int ACT>
-static int launch_silu_mul(void* out, const void* gu, int rows, int inter, cudaStream_t stream) {
+static int launch_silu_mul(void* out, const void* gu, int rows, int inter, cudaStream_t stream, float limit = 0.f) {
   if (rows <= 0 || inter <= 0) return 0;
   if (rows > 65535) return EK_ERR_ARG;
   if (sizeof(T) == 2 && inter % 8 == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)gu % 16) == 0) {
     dim3 wide((inter / 8 + 255) / 256, rows);
-    silu_mul_wide_kernel<ACT><<<wide, 256, 0, stream>>>((bf16*)out, (const bf16*)gu, inter);
+    silu_mul_wide_kernel<ACT><<<wide, 256, 0, stream>>>((bf16*)out, (const bf16*)gu, inter, limit);
     EK_RETURN_LAUNCH_STATUS();
   }
   const bool vec = inter % 4 == 0 && ((uintptr_t)out % 8) == 0 && ((uintptr_t)gu % 8) == 0;
   const int per_thread = vec ? 4 : 1;
   dim3 grid((inter / per_thread + 255) / 256 + (inter % per_thread ? 1 : 0), rows);
-  if (vec) silu_mul_kernel<T, true, ACT><<<grid, 256, 0, stream>>>((T*)out, (const T*)gu, inter);
-  else silu_mul_kernel<T, false, ACT><<<grid, 256, 0, stream>>>((T*)out, (const T*)gu, inter);
+  if (vec) silu_mul_kernel<T, true, ACT><<<grid, 256, 0, stream>>>((T*)out, (const T*)gu, inter, limit);
+  else silu_mul_kernel<T, false, ACT><<<grid, 256, 0, stream>>>((T*)out, (const T*)gu, inter, limit);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -608,11 +621,12 @@ using namespace ek;
                                      cudaStream_t stream) {                                     \
     return launch_silu_mul<T, 0>(out, gu, rows, inter, stream);                                 \
   }                                                                                             \
-  /* act 0: silu, 1: gelu (tanh form) */                                                        \
+  /* act 0: silu, 1: gelu (tanh form), 2: the clamped gate with `limit` */                     \
   EK_EXPORT int ek_act_mul_##SUFFIX(void* out, const void* gu, int rows, int inter, int act,    \
-                                    cudaStream_t stream) {                                      \
+                                    float limit, cudaStream_t stream) {                         \
     if (act == 0) return launch_silu_mul<T, 0>(out, gu, rows, inter, stream);                   \
     if (act == 1) return launch_silu_mul<T, 1>(out, gu, rows, inter, stream);                   \
+    if (act == 2 && limit > 0.f) return launch_silu_mul<T, 2>(out, gu, rows, inter, stream, limit); \
     return EK_ERR_ARG;                                                                          \
   }
 

@@ -60,6 +60,7 @@ struct TcParams {
   int k_blocks_per_split;
   int swiglu_half;      // SwiGLU: second-half row offset in the weight matrix (I)
   int gate_gelu;        // the gate's activation: 0 SiLU, 1 the tanh form of GELU
+  float gate_limit;     // > 0: the clamped form instead (gate_clamped_fast)
   float* partials;      // split-K scratch [tile][split][BN][128]
   unsigned int* tickets;
   int* status;          // 0, or the code of the first wait that timed out
@@ -448,8 +449,13 @@ gemm_tc_bf16_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
           if (EPI == TC_EPI_SWIGLU) {
             n_out = tile_p * 64 + r0;
             n_limit = prm.swiglu_half;
-            acc.x = gate_fast(acc.x, prm.gate_gelu) * up.x; acc.y = gate_fast(acc.y, prm.gate_gelu) * up.y;
-            acc.z = gate_fast(acc.z, prm.gate_gelu) * up.z; acc.w = gate_fast(acc.w, prm.gate_gelu) * up.w;
+            if (prm.gate_limit > 0.f) {
+              acc.x = gate_clamped_fast(acc.x, up.x, prm.gate_limit); acc.y = gate_clamped_fast(acc.y, up.y, prm.gate_limit);
+              acc.z = gate_clamped_fast(acc.z, up.z, prm.gate_limit); acc.w = gate_clamped_fast(acc.w, up.w, prm.gate_limit);
+            } else {
+              acc.x = gate_fast(acc.x, prm.gate_gelu) * up.x; acc.y = gate_fast(acc.y, prm.gate_gelu) * up.y;
+              acc.z = gate_fast(acc.z, prm.gate_gelu) * up.z; acc.w = gate_fast(acc.w, prm.gate_gelu) * up.w;
+            }
           } else {
             n_out = tile_p * kTcBM + r0;
             n_limit = prm.rows_p;
@@ -632,8 +638,13 @@ gemm_tc_bf16_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
         fetch(c0, v);
         if (EPI == TC_EPI_SWIGLU && !SWAP) {
           fetch(c0 + BN / 2, u);               // the matching up columns
+          if (prm.gate_limit > 0.f) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = gate_fast(v[i], prm.gate_gelu) * u[i];
+            for (int i = 0; i < 16; ++i) v[i] = gate_clamped_fast(v[i], u[i], prm.gate_limit);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] = gate_fast(v[i], prm.gate_gelu) * u[i];
+          }
         }
         if (EPI == TC_EPI_SWIGLU && SWAP) {
           // rows 64..127 hold the up rows of the gate rows 0..63: pass them through shared memory
@@ -644,8 +655,13 @@ gemm_tc_bf16_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
           }
           __syncthreads();
           if (row < 64) {
+            if (prm.gate_limit > 0.f) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) v[i] = gate_fast(v[i], prm.gate_gelu) * xch[row * 16 + i];
+              for (int i = 0; i < 16; ++i) v[i] = gate_clamped_fast(v[i], xch[row * 16 + i], prm.gate_limit);
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i) v[i] = gate_fast(v[i], prm.gate_gelu) * xch[row * 16 + i];
+            }
           }
         }
         if (SWAP) {
@@ -772,7 +788,8 @@ static int launch_tc(const CUtensorMap& mp, const CUtensorMap& mq, const TcParam
 }  // namespace ek
 
 // out[M, N] = x[M, K] . w[N, K]^T  (epilogue 0/1) or out[M, N/2] = act(x.wg^T) * (x.wu^T) with w =
-// [gate rows; up rows] (epilogue 2: act = SiLU; 3: the tanh form of GELU).  Epilogue 4 (swapped form only)
+// [gate rows; up rows] (epilogue 2: act = SiLU; 3: the tanh form of GELU).  gate_limit > 0 (epilogue 2): the
+// clamped form of the gate instead (gate_clamped_fast).  Epilogue 4 (swapped form only)
 // is epilogue 0 computed by the instantiation that also holds the extended q/k/v epilogue.  swap != 0: weights fill the 128-row MMA side (for
 // 1..64 rows of x); k_split blocks share a tile's K: as a cluster if `cluster` != 0 and k_split is
 // at most 8, else through `partials` (at least tiles * k_split * bn * 128 floats) and zeroed
@@ -864,8 +881,10 @@ EK_EXPORT int ek_gemm_tc_bf16(void* out, const void* x, const void* w, int M, in
                               float* partials, unsigned int* tickets, long long partial_floats,
                               int n_tickets, const float* ss_in, int ss_tiles, int norm_size, float eps,
                               float* residual, int ld_residual, const float* next_gain, float* ss_out,
-                              int* status, cudaStream_t stream) {
-  return gemm_tc_run(ek::TcParams{}, out, x, w, M, N, K, ldx, ldw, ldo, epilogue, swap, k_split, cluster,
+                              float gate_limit, int* status, cudaStream_t stream) {
+  ek::TcParams extras{};
+  extras.gate_limit = epilogue == ek::TC_EPI_SWIGLU ? gate_limit : 0.f;
+  return gemm_tc_run(extras, out, x, w, M, N, K, ldx, ldw, ldo, epilogue, swap, k_split, cluster,
                      partials, tickets, partial_floats, n_tickets, ss_in, ss_tiles, norm_size, eps,
                      residual, ld_residual, next_gain, ss_out, status, stream);
 }

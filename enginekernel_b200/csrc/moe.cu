@@ -6,7 +6,9 @@
 //             `keep` best groups can be chosen; the `top` largest of those; weights = chosen
 //             scores / (their sum + 1e-20) * scale.  A warp a token.  `among_chosen`: the weights are
 //             the softmax over the chosen logits alone (times scale), taken from the logits with the
-//             chosen maximum off, so that no score can vanish against an unchosen expert's.
+//             chosen maximum off, so that no score can vanish against an unchosen expert's.  `mode` 2: scores
+//             are sigmoids of the logits, each for itself; the weights are the chosen scores times scale,
+//             not divided by their sum.
 //   plan      the (token, choice) pairs sorted by expert, and the row tiles of every expert's
 //             stretch, made on the device: the host never sees who chose what.
 //   expert product  out[row] = f(x[row] . W_e^T) over the tiles of the plan: FFMA with 32-bit
@@ -17,7 +19,10 @@
 //             scatters 32-bit rows by pair.  `gated` up form: the expert's weight rows alternate
 //             gate, up, gate, up ...; column pair (2c, 2c + 1) of the product gives out[c] =
 //             act(gate) * up from the 32-bit sums (N counts the weight rows, the output has N / 2).
-//   combine   out[t] = sum over the token's choices, in the order they were chosen.
+//             `row_weight` (up form): a pair's weight multiplies its row of the product before the activation,
+//             which is the product of the weighted input; `limit` belongs to the clamped activation.
+//   combine   out[t] = sum over the token's choices, in the order they were chosen (+ add[t], the result of an
+//             expert that every token shares).
 #include "common.cuh"
 
 namespace ek {
@@ -37,7 +42,9 @@ constexpr int kRouteWarps = 4;
 __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
                  const float* __restrict__ logits, int n_tokens, int E, int n_groups, int keep, int top,
-                 float scale, int among_chosen) {
+                 float scale, int mode) {
+  // mode 0: softmax scores, divided by the chosen ones' sum; 1: softmax over the chosen; 2: sigmoids as they are
+  const bool among_chosen = mode != 0;          // (candidates are compared by their logits)
   extern __shared__ float route_s[];            // per warp: scores [E], candidates [E], groups [n_groups]
   pdl_launch_dependents();
   pdl_wait();
@@ -95,6 +102,14 @@ moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
       cand[bi] = shut;
     }
     __syncwarp();
+  }
+  if (mode == 2) {
+    __syncwarp();
+    for (int k = lane; k < top; k += 32) {
+      const float x = z[sel_expert[(size_t)t * top + k]];
+      sel_weight[(size_t)t * top + k] = scale / (1.f + expf(-x));
+    }
+    return;
   }
   if (among_chosen) {                           // softmax over the chosen logits: the first chosen is the largest
     __syncwarp();
@@ -157,13 +172,22 @@ moe_plan_kernel(int* __restrict__ sorted_pair, int* __restrict__ tiles, int* __r
   }
 }
 
-constexpr int ACT_RELU2 = 1, ACT_SILU = 2, ACT_GELU_TANH = 3;      // 0: none
+constexpr int ACT_RELU2 = 1, ACT_SILU = 2, ACT_GELU_TANH = 3, ACT_CLAMPED = 4;      // 0: none
 
 __device__ __forceinline__ float activate(float z, int act) {
   if (act == ACT_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
   if (act == ACT_SILU) return z / (1.f + expf(-z));
   if (act == ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z;
+}
+
+// act(gate) * up; the clamped form is g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+__device__ __forceinline__ float gated_value(float gate, float up, int act, float limit) {
+  if (act == ACT_CLAMPED) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+  }
+  return activate(gate, act) * up;
 }
 
 // grid (max tiles, column tiles).  UP: a[row] = x[pair / top], out T [sorted row][N] = act(.).
@@ -173,7 +197,7 @@ __global__ void __launch_bounds__(256)
 moe_expert_product_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __restrict__ w,
                           const int* __restrict__ tiles, const int* __restrict__ n_tiles,
                           const int* __restrict__ sorted_pair, const float* __restrict__ pair_weight,
-                          int top, int N, int K, int act, int gated) {
+                          int top, int N, int K, int act, int gated, float limit) {
   constexpr int BM = kTileRows, BN = 64, BK = 16, TM = 4, TN = 4, PAD = 4;
   __shared__ __align__(16) float As[BK][BM + PAD];
   __shared__ __align__(16) float Ws[BK][BN + PAD];
@@ -228,18 +252,19 @@ moe_expert_product_kernel(void* __restrict__ out_, const T* __restrict__ a, cons
   for (int i = 0; i < TM; ++i) {
     const int r = ty * TM + i;
     if (r >= rows) continue;
+    const float rw = UP && pair_weight != nullptr ? pair_weight[pair_s[r]] : 1.f;
 #pragma unroll
     for (int j = 0; j < TN; ++j) {
       const int gn = n0 + tx * TN + j;
       if (gn >= N) continue;
       if (UP && gated) {                          // columns (gn, gn + 1) = (gate, up); N is even
         if (!(j & 1)) ((T*)out_)[(size_t)(row0 + r) * (N / 2) + gn / 2] =
-            from_f<T>(activate(acc[i][j], act) * acc[i][j + 1]);
+            from_f<T>(gated_value(acc[i][j] * rw, acc[i][j + 1] * rw, act, limit));
       } else if (UP) {
-        ((T*)out_)[(size_t)(row0 + r) * N + gn] = from_f<T>(activate(acc[i][j], act));
+        ((T*)out_)[(size_t)(row0 + r) * N + gn] = from_f<T>(activate(acc[i][j] * rw, act));
       } else {
         const int p = pair_s[r];
-        ((float*)out_)[(size_t)p * N + gn] = acc[i][j] * pair_weight[p];
+        ((float*)out_)[(size_t)p * N + gn] = acc[i][j] * (pair_weight != nullptr ? pair_weight[p] : 1.f);
       }
     }
   }
@@ -282,7 +307,7 @@ __global__ void __launch_bounds__(256)
 moe_expert_product_tc_kernel(void* __restrict__ out_, const bf16* __restrict__ a, const bf16* __restrict__ w,
                              const int* __restrict__ tiles, const int* __restrict__ n_tiles,
                              const int* __restrict__ sorted_pair, const float* __restrict__ pair_weight,
-                             int top, int N, int K, int act, int gated) {
+                             int top, int N, int K, int act, int gated, float limit) {
   constexpr int BM = kTileRows, BN = kTcCols, BK = kTcK, LD = kTcLd, STAGES = kTcStages;
   extern __shared__ __align__(16) unsigned char tc_smem[];
   typedef bf16 (*Tile)[LD];
@@ -369,14 +394,14 @@ moe_expert_product_tc_kernel(void* __restrict__ out_, const bf16* __restrict__ a
       const int r = wm * 32 + i * 16 + g + half * 8;
       if (r >= rows) continue;
       const int p = pair_s[r];
-      const float pw = UP ? 1.f : pair_weight[p];
+      const float pw = pair_weight != nullptr ? pair_weight[p] : 1.f;
       if (UP && gated) {                          // a lane's two neighbouring columns are (gate, up)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int gn = n0 + wn * 32 + j * 8 + tq * 2;
           if (gn + 1 < N)
             ((bf16*)out_)[(size_t)(row0 + r) * (N / 2) + gn / 2] =
-                __float2bfloat16_rn(activate(acc[i][j][half * 2], act) * acc[i][j][half * 2 + 1]);
+                __float2bfloat16_rn(gated_value(acc[i][j][half * 2] * pw, acc[i][j][half * 2 + 1] * pw, act, limit));
         }
         continue;
       }
@@ -387,7 +412,7 @@ moe_expert_product_tc_kernel(void* __restrict__ out_, const bf16* __restrict__ a
           const int gn = n0 + wn * 32 + j * 8 + tq * 2 + c;
           if (gn >= N) continue;
           const float v = acc[i][j][half * 2 + c];
-          if (UP) ((bf16*)out_)[(size_t)(row0 + r) * N + gn] = __float2bfloat16_rn(activate(v, act));
+          if (UP) ((bf16*)out_)[(size_t)(row0 + r) * N + gn] = __float2bfloat16_rn(activate(v * pw, act));
           else ((float*)out_)[(size_t)p * N + gn] = v * pw;
         }
     }
@@ -396,13 +421,14 @@ moe_expert_product_tc_kernel(void* __restrict__ out_, const bf16* __restrict__ a
 // out[t, :] = sum_k pair_out[t * top + k, :], k ascending.
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ pair_out, int top,
-                                   int width) {
+                                   int width, const T* __restrict__ add) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float a = 0.f;
     for (int k = 0; k < top; ++k) a += pair_out[(t * top + k) * width + i];
+    if (add) a += to_f<T>(add[t * width + i]);
     out[t * width + i] = from_f<T>(a);
   }
 }
@@ -412,12 +438,12 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
 EK_EXPORT int ek_moe_tile_rows() { return ek::kTileRows; }
 
 EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logits, int n_tokens, int E,
-                           int n_groups, int keep, int top, float scale, int among_chosen,
+                           int n_groups, int keep, int top, float scale, int mode,
                            cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
-      top > keep * (E / n_groups))
+      top > keep * (E / n_groups) || mode < 0 || mode > 2 || (mode == 2 && keep < n_groups))
     return EK_ERR_ARG;
   const size_t smem = (size_t)kRouteWarps * (2 * E + n_groups) * sizeof(float);
   if (smem > 200 * 1024) return EK_ERR_ARG;
@@ -426,7 +452,7 @@ EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logi
     if (e != cudaSuccess) return (int)e;
   }
   moe_route_kernel<<<(n_tokens + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, stream>>>(
-      sel_expert, sel_weight, logits, n_tokens, E, n_groups, keep, top, scale, among_chosen);
+      sel_expert, sel_weight, logits, n_tokens, E, n_groups, keep, top, scale, mode);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -442,10 +468,10 @@ EK_EXPORT int ek_moe_plan(int* sorted_pair, int* tiles, int* n_tiles, const int*
 // The tensor-core forms: bfloat16, K a multiple of 8, operands on 16-byte boundaries.
 EK_EXPORT int ek_moe_expert_up_tc(void* out, const void* x, const void* w, const int* tiles, const int* n_tiles,
                                   const int* sorted_pair, int max_tiles, int top, int N, int K, int act,
-                                  int gated, cudaStream_t stream) {
+                                  int gated, float limit, const float* row_weight, cudaStream_t stream) {
   using namespace ek;
   if (max_tiles <= 0) return 0;
-  if (gated && N % 2) return EK_ERR_ARG;
+  if ((gated && N % 2) || (act == ACT_CLAMPED && !(gated && limit > 0.f))) return EK_ERR_ARG;
   if (N <= 0 || K <= 0 || K % 8 || top <= 0 || (N + 127) / 128 > 65535 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return EK_ERR_ARG;
   dim3 grid(max_tiles, (N + 127) / 128);
@@ -453,7 +479,7 @@ EK_EXPORT int ek_moe_expert_up_tc(void* out, const void* x, const void* w, const
                                        (int)kTcSmem);
   if (e != cudaSuccess) return (int)e;
   moe_expert_product_tc_kernel<true><<<grid, 256, kTcSmem, stream>>>(out, (const bf16*)x, (const bf16*)w, tiles, n_tiles,
-                                                              sorted_pair, nullptr, top, N, K, act, gated);
+                                                              sorted_pair, row_weight, top, N, K, act, gated, limit);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -469,21 +495,23 @@ EK_EXPORT int ek_moe_expert_down_tc(float* out, const void* a, const void* w, co
                                        (int)kTcSmem);
   if (e != cudaSuccess) return (int)e;
   moe_expert_product_tc_kernel<false><<<grid, 256, kTcSmem, stream>>>(out, (const bf16*)a, (const bf16*)w, tiles, n_tiles,
-                                                               sorted_pair, pair_weight, 1, N, K, 0, 0);
+                                                               sorted_pair, pair_weight, 1, N, K, 0, 0, 0.f);
   EK_RETURN_LAUNCH_STATUS();
 }
 
 #define EK_INSTANTIATE(SUFFIX, T)                                                                     \
   EK_EXPORT int ek_moe_expert_up_##SUFFIX(void* out, const void* x, const void* w, const int* tiles,  \
                                           const int* n_tiles, const int* sorted_pair, int max_tiles,  \
-                                          int top, int N, int K, int act, int gated,                  \
-                                          cudaStream_t stream) {                                      \
+                                          int top, int N, int K, int act, int gated, float limit,     \
+                                          const float* row_weight, cudaStream_t stream) {             \
     using namespace ek;                                                                               \
     if (max_tiles <= 0) return 0;                                                                     \
-    if (N <= 0 || K <= 0 || top <= 0 || (N + 63) / 64 > 65535 || (gated && N % 2)) return EK_ERR_ARG; \
+    if (N <= 0 || K <= 0 || top <= 0 || (N + 63) / 64 > 65535 || (gated && N % 2) ||         \
+        (act == ACT_CLAMPED && !(gated && limit > 0.f)))                                              \
+      return EK_ERR_ARG;                                                                              \
     dim3 grid(max_tiles, (N + 63) / 64);                                                              \
     moe_expert_product_kernel<T, true><<<grid, 256, 0, stream>>>(                                     \
-        out, (const T*)x, (const T*)w, tiles, n_tiles, sorted_pair, nullptr, top, N, K, act, gated);  \
+        out, (const T*)x, (const T*)w, tiles, n_tiles, sorted_pair, row_weight, top, N, K, act, gated, limit); \
     EK_RETURN_LAUNCH_STATUS();                                                                        \
   }                                                                                                   \
   EK_EXPORT int ek_moe_expert_down_##SUFFIX(float* out, const void* a, const void* w, const int* tiles, \
@@ -495,13 +523,13 @@ EK_EXPORT int ek_moe_expert_down_tc(float* out, const void* a, const void* w, co
     if (N <= 0 || K <= 0 || (N + 63) / 64 > 65535) return EK_ERR_ARG;                                 \
     dim3 grid(max_tiles, (N + 63) / 64);                                                              \
     moe_expert_product_kernel<T, false><<<grid, 256, 0, stream>>>(                                    \
-        out, (const T*)a, (const T*)w, tiles, n_tiles, sorted_pair, pair_weight, 1, N, K, 0, 0);      \
+        out, (const T*)a, (const T*)w, tiles, n_tiles, sorted_pair, pair_weight, 1, N, K, 0, 0, 0.f); \
     EK_RETURN_LAUNCH_STATUS();                                                                        \
   }                                                                                                   \
   EK_EXPORT int ek_moe_combine_##SUFFIX(void* out, const float* pair_out, int n_tokens, int top,      \
-                                        int width, cudaStream_t stream) {                             \
+                                        int width, const void* add, cudaStream_t stream) {            \
     if (n_tokens <= 0) return 0;                                                                      \
-    ek::moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>((T*)out, pair_out, top, width);           \
+    ek::moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>((T*)out, pair_out, top, width, (const T*)add); \
     EK_RETURN_LAUNCH_STATUS();                                                                        \
   }
 

@@ -18,6 +18,8 @@
 //   xgate_scan       a, b and the running maximum of the matrix memory (a warp a head, 32 tokens a pass)
 //   decay_scan       the recurrence; reads and writes S in the state
 //   ssm_out          (o + D x) silu(z), RMS norm in equal parts, weight -> activation type
+//   norm_gate_out    RMS norm over all heads together, weight, sigmoid gate -> activation type (a matrix state
+//                    whose decays are one constant per head: decay_scan with a and b the same for every token)
 //   xlstm_out        o / (max(|n.q|, exp(-m)) + 1e-6), RMS norm per head, weight, sigmoid gate
 // and a recurrence with a decay per CHANNEL and no matrix state (a gated linear recurrent unit):
 //   lru_gates        both gates from block-diagonal products, the decay and the gated input
@@ -455,6 +457,7 @@ constexpr int kScanFloats = 2048;    // values of keys (and of queries) fetched 
 // grid (sequences, heads, column tiles).  RPL rows of a column a lane: lane l holds rows 32 g + 4 l + c
 // (g < RPL / 4, c < 4), so that the 8 lanes of a column read 128 neighbouring bytes of a key at a time.
 // S of a slot: state[((h * C + j) * DK + i], DK = 8 RPL rows (keys padded with zeros), C = dv + ones_col columns.
+// `ab_stride`: values of a (and b) from token to token - the heads, or 0 where they are the same for every token.
 // Column dv (with ones_col) has v = 1: it carries n_t = a n + b k and gives n.q.
 // Tokens come 2048 / DK at a time: while one portion is worked through from shared memory, the next one's
 // keys, queries, values and gates are already on their way into registers.
@@ -465,7 +468,7 @@ decay_scan_kernel(float* __restrict__ out, int out_stride, const float* __restri
                   const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ state,
                   size_t slot_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ positions,
                   const int* __restrict__ token_slot, int heads, int kv_heads, int dk, int dv, int ones_col,
-                  int write_state) {
+                  int write_state, int ab_stride) {
   constexpr int DK = 8 * RPL, G4 = RPL / 4, DK4 = DK / 4;
   constexpr int CH = kScanFloats / DK;                       // tokens a portion: 64, 32, 16 or 8
   constexpr int NV4 = kScanFloats / 4 / kScanThreads;        // float4 of keys (of queries) a thread fetches
@@ -527,8 +530,8 @@ decay_scan_kernel(float* __restrict__ out, int out_stride, const float* __restri
     }
     a_r = 1.f, b_r = 0.f;                        // tokens past the end leave S as it is
     if (tid < nc) {
-      a_r = a[((size_t)start + c0 + tid) * heads + h];
-      b_r = b[((size_t)start + c0 + tid) * heads + h];
+      a_r = a[((size_t)start + c0 + tid) * ab_stride + h];
+      b_r = b[((size_t)start + c0 + tid) * ab_stride + h];
     }
   };
   fetch(0);
@@ -814,9 +817,10 @@ EK_EXPORT int ek_decay_scan(float* out, int out_stride, const float* q, int q_st
                             const float* v, int v_stride, const float* a, const float* b, float* state,
                             long long slot_stride, const int* cu_seqlens, const int* positions,
                             const int* token_slot, int n_seqs, int heads, int kv_heads, int dk, int dv,
-                            int ones_col, int write_state, cudaStream_t stream) {
+                            int ones_col, int write_state, int ab_stride, cudaStream_t stream) {
   using namespace ek;
   if (n_seqs <= 0) return 0;
+  if (ab_stride != 0 && ab_stride != heads) return EK_ERR_ARG;
   const int rows = ek_decay_scan_rows(dk);
   if (!rows || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dv <= 0 || heads > 65535 || slot_stride % 4 ||
       ((uintptr_t)state & 15))
@@ -827,8 +831,40 @@ EK_EXPORT int ek_decay_scan(float* out, int out_stride, const float* q, int q_st
               : rows == 128 ? decay_scan_kernel<16> : decay_scan_kernel<32>;
   return (int)launch_pdl(kernel, grid, dim3(kScanThreads), 0, stream, out, out_stride, q, q_stride, k, k_stride, v,
                          v_stride, a, b, state, (size_t)slot_stride, cu_seqlens, positions, token_slot, heads,
-                         kv_heads, dk, dv, ones_col ? 1 : 0, write_state);
+                         kv_heads, dk, dv, ones_col ? 1 : 0, write_state, ab_stride);
 }
+
+// y[t, c] = rms-normed over all `inner` channels o * w[c] * sigmoid(proj[t, col_g + c]).  A block a token.
+namespace ek {
+template <typename T>
+__global__ void __launch_bounds__(1024)
+norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float* __restrict__ proj, int proj_stride,
+                     int col_g, const float* __restrict__ w, float eps, const int* __restrict__ positions, int inner) {
+  __shared__ float scratch[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  if (positions[t] < 0) return;
+  const float* row = o + t * inner;
+  const float* gate = proj + t * proj_stride + col_g;
+  float u[kOutKeep], ss = 0.f;
+#pragma unroll
+  for (int m = 0; m < kOutKeep; ++m) {           // the first values of a thread wait in registers
+    const int i = threadIdx.x + m * blockDim.x;
+    u[m] = i < inner ? row[i] : 0.f;
+    ss += u[m] * u[m];
+  }
+  for (int i = threadIdx.x + kOutKeep * blockDim.x; i < inner; i += blockDim.x) ss += row[i] * row[i];
+  const float rstd = rsqrtf(block_sum(ss, scratch) / (float)inner + eps);
+#pragma unroll
+  for (int m = 0; m < kOutKeep; ++m) {
+    const int i = threadIdx.x + m * blockDim.x;
+    if (i < inner) y[t * inner + i] = from_f<T>(u[m] * rstd * w[i] * sigmoid_f(gate[i]));
+  }
+  for (int i = threadIdx.x + kOutKeep * blockDim.x; i < inner; i += blockDim.x)
+    y[t * inner + i] = from_f<T>(row[i] * rstd * w[i] * sigmoid_f(gate[i]));
+}
+}  // namespace ek
 
 #define EK_INSTANTIATE(SUFFIX, T)                                                                              \
   EK_EXPORT int ek_ssm_out_##SUFFIX(void* y, const float* o, const float* x, int x_stride, const float* proj,  \
@@ -843,6 +879,15 @@ EK_EXPORT int ek_decay_scan(float* out, int out_stride, const float* q, int q_st
     return (int)ek::launch_pdl(ek::ssm_out_kernel<T>, dim3(n_tokens, parts), dim3(threads), 0, stream, (T*)y,  \
                                o, x, x_stride, proj, proj_stride, col_z, d_skip, w, eps, positions, inner,     \
                                vdim, parts);                                                                   \
+  }                                                                                                            \
+  EK_EXPORT int ek_norm_gate_out_##SUFFIX(void* y, const float* o, const float* proj, int proj_stride, int col_g, \
+                                          const float* w, float eps, const int* positions, int n_tokens,       \
+                                          int inner, cudaStream_t stream) {                                    \
+    if (n_tokens <= 0) return 0;                                                                               \
+    if (inner <= 0) return EK_ERR_ARG;                                                                         \
+    const int threads = inner >= 4096 ? 1024 : inner <= 256 ? 64 : (inner / 4 + 31) / 32 * 32;                 \
+    return (int)ek::launch_pdl(ek::norm_gate_out_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (T*)y, o, \
+                               proj, proj_stride, col_g, w, eps, positions, inner);                            \
   }                                                                                                            \
   EK_EXPORT int ek_xlstm_out_##SUFFIX(void* y, const float* o, const float* m_run, const float* proj,          \
                                       int proj_stride, int col_g, const float* w, float eps, float q_scale,    \

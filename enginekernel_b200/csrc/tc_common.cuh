@@ -22,6 +22,13 @@ __device__ __forceinline__ float gate_fast(float x, int gelu_tanh) {
   return __fdividef(x, 1.f + __expf(-z));
 }
 
+// A gated feed-forward whose halves are clamped: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(1.702 g) (u + 1).
+__device__ __forceinline__ float gate_clamped_fast(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
+}
+
 // ---------------------------------------------------------------------------- PTX wrappers
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
   return (uint32_t)__cvta_generic_to_shared(p);

@@ -65,7 +65,7 @@ def _need(cond, msg):
         raise KernelError(msg)
 
 
-def _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, new_keys_only):
+def _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, new_keys_only, chunk=None):
     """While a launch record is active: what an attention launch has to read and compute.  Reads
     the positions back (a synchronisation, which is why it is done only then).  Keys and values:
     for single tokens every visible key of every token; for prompts (``new_keys_only``) each
@@ -76,6 +76,8 @@ def _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, win
     visible = torch.clamp(pos + 1, min=0)
     if window:
         visible = torch.clamp(visible, max=int(window))
+    if chunk:
+        visible = torch.where(pos >= 0, pos % int(chunk) + 1, visible)
     keys = int(visible.sum().item())
     live = int((pos >= 0).sum().item())
     size = q.element_size()
@@ -94,8 +96,9 @@ _scale_f32 = Function("elementwise", "ek_scale_f32", [_P, c_longlong, c_float, _
 _rmsnorm = _per_dtype("elementwise", "ek_rmsnorm",
                       [_P, _P, _P, _P, _P, c_float, c_int, c_int, c_int, _P])
 _add_residual = _per_dtype("elementwise", "ek_add_residual", [_P, _P, c_longlong, _P])
-_act_mul = _per_dtype("elementwise", "ek_act_mul", [_P, _P, c_int, c_int, c_int, _P])
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+_act_mul = _per_dtype("elementwise", "ek_act_mul", [_P, _P, c_int, c_int, c_int, c_float, _P])
+# "clamped": min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1)
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
 
 
 def embed(resid, table, ids, n_tokens, scale=1.0, pos_table=None, positions=None, accumulate=False):
@@ -214,10 +217,12 @@ def silu_mul(out, gu, n_rows=None):
     act_mul(out, gu, "silu", n_rows)
 
 
-def act_mul(out, gu, activation="silu", n_rows=None):
+def act_mul(out, gu, activation="silu", n_rows=None, limit=0.0):
     """out[r, i] = act(gu[r, i]) * gu[r, I + i] for gu of width 2I; ``activation`` is ``"silu"`` or
-    ``"gelu_tanh"`` (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))))."""
+    ``"gelu_tanh"`` (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))); ``"clamped"`` with a positive
+    ``limit``: with g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(1.702 g') (u' + 1)."""
     _need_cuda(out, gu)
+    _need(activation != "clamped" or limit > 0, "act_mul: the clamped gate needs a positive limit")
     _need(activation in GATE_ACTIVATIONS, f"act_mul: no activation {activation!r}")
     inter = gu.shape[-1] // 2
     _need(gu.shape[-1] == 2 * inter and out.shape[-1] == inter and out.dtype == gu.dtype,
@@ -229,7 +234,7 @@ def act_mul(out, gu, activation="silu", n_rows=None):
     for r0 in range(0, rows, 65535):
         r1 = min(rows, r0 + 65535)
         _act_mul[gu.dtype](_ptr(out[r0:]), _ptr(gu[r0:]), r1 - r0, inter, GATE_ACTIVATIONS[activation],
-                           _stream())
+                           float(limit), _stream())
 
 
 _embed_pair = _per_dtype("elementwise", "ek_embed_pair",
@@ -314,6 +319,89 @@ def bias_act(out, x, bias=None, activation=None, col0=0, n_rows=None):
                          width, n, ROW_ACTIVATIONS[activation], _stream())
 
 
+# ------------------------------------------------------------------ dynamic tanh, averages over the depth
+_dynamic_tanh = _per_dtype("depth", "ek_dynamic_tanh",
+                           [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P])
+_depth_join = _per_dtype("depth", "ek_depth_join",
+                         [_P, _P, _P, _P, c_longlong, _P, c_int, c_int, c_float, _P, _P, _P, _P, _P, c_float, c_float,
+                          _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P])
+
+
+def _tanh_norm_args(y, norm, hidden, name):
+    """(y, alpha, w, b) pointers of one reader; ``norm`` is (alpha [1], w [hidden], b [hidden]) in 32-bit."""
+    if y is None:
+        return [None] * 4
+    alpha, w, b = norm
+    _need_cuda(y, alpha, w, b)
+    _need(y.is_contiguous() and y.shape[-1] == hidden, f"{name}: packed rows of the stream's width")
+    for t, n in ((alpha, 1), (w, hidden), (b, hidden)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n,
+              f"{name}: 32-bit alpha [1], weight and shift of the stream's width")
+    return [_ptr(t) for t in (y, alpha, w, b)]
+
+
+def dynamic_tanh(y, stream, norm, second=None, second_norm=None, add=None, rows=None, n_rows=None, write_back=True):
+    """y = tanh(alpha x) w + b with ``norm`` = (alpha, w, b) in 32-bit, and the same of ``second_norm`` into
+    ``second``; x = stream [+ add], the stream updated in place when ``write_back``.  ``rows`` (int32) picks
+    stream rows (and the same rows of ``add``)."""
+    _need_cuda(y, stream, second, add, rows)
+    hidden = stream.shape[-1]
+    _need(stream.dtype == torch.float32 and stream.is_contiguous(), "dynamic_tanh: a 32-bit stream")
+    _need(add is None or (add.dtype == y.dtype and add.is_contiguous() and add.shape[-1] == hidden),
+          "dynamic_tanh: add has y's type and the stream's width")
+    _need(second is None or second.dtype == y.dtype, "dynamic_tanh: both readers have one type")
+    n = n_rows if n_rows is not None else (rows.numel() if rows is not None else stream.shape[0])
+    if lib.recording():
+        lib.annotate(bytes=n * hidden * (4 + y.element_size() * ((1 if second is None else 2) + (0 if add is None else 1))
+                                         + (4 if add is not None and write_back else 0)))
+    _dynamic_tanh[y.dtype](*_tanh_norm_args(y, norm, hidden, "dynamic_tanh"),
+                           *_tanh_norm_args(second, second_norm, hidden, "dynamic_tanh"), _ptr(stream), _ptr(add),
+                           _ptr(rows), n, hidden, 1 if write_back else 0, _stream())
+
+
+def depth_join(x_next, x, first, kept, n, depth, mult, a, gate_a, f=None, gate_f=None, bias_a=None, pair=None,
+               keep=True, y1=None, norm1=None, y2=None, norm2=None, n_rows=None):
+    """What stands between two layers.  r = x + mult (sigmoid(z_a + b_a) a + sigmoid(z_f + b_f) f), kept as entry
+    n - 1 of ``kept`` [entries, rows, hidden] when ``keep``; x_next = sum_(j < n) depth[j] X_j + depth[n] r with
+    X_0 = ``first`` and X_j = kept[j - 1]; y1, y2 = tanh norms of x_next (``norm1``, ``norm2`` as in
+    :func:`dynamic_tanh`, absent: not wanted).  ``gate_a`` = (z_a [rows, hidden], b_a [hidden] 32-bit), ``gate_f`` alike;
+    ``f`` absent: no second sublayer.  ``bias_a`` (32-bit) is added to ``a``; ``pair`` = (b, gain_a, gain_b, eps,
+    weight) instead: the first result is weight (a / rms(a) gain_a + b / rms(b) gain_b)."""
+    _need_cuda(x_next, x, first, kept, depth, a, f, bias_a, y1, y2)
+    hidden = x.shape[-1]
+    rows = n_rows if n_rows is not None else x.shape[0]
+    for t in (x_next, x, first):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape[-1] == hidden and t.shape[0] >= rows,
+              "depth_join: 32-bit streams [rows, hidden]")
+    _need(depth.dtype == torch.float32 and depth.is_contiguous() and depth.numel() == n + 1,
+          "depth_join: one 32-bit weight per earlier result and one for this one")
+    entries = n if keep else n - 1
+    _need(entries == 0 or (kept is not None and kept.dtype == torch.float32 and kept.is_contiguous() and kept.dim() == 3
+                           and kept.shape[0] >= entries and kept.shape[1] >= rows and kept.shape[2] == hidden),
+          "depth_join: room for the kept results [entries, rows, hidden]")
+    (za, ba), (zf, bf) = gate_a, gate_f if f is not None else (None, None)
+    b = gain_a = gain_b = None
+    eps = weight = 0.0
+    if pair is not None:
+        b, gain_a, gain_b, eps, weight = pair
+    for t in (a, b, za, f, zf, y1, y2):
+        _need(t is None or (t.is_cuda and t.dtype == a.dtype and t.is_contiguous() and t.shape[-1] == hidden),
+              "depth_join: results and gate products of one type and the stream's width")
+    for t in (ba, bf, bias_a, gain_a, gain_b):
+        _need(t is None or (t.is_cuda and t.dtype == torch.float32 and t.is_contiguous() and t.numel() == hidden),
+              "depth_join: 32-bit vectors of the stream's width")
+    if lib.recording():
+        # x, X_0 .. X_(n-1), x' and r; the results and gate products; the readers' rows (X_0 is x itself in the first layer)
+        streams = (0 if x.data_ptr() == first.data_ptr() else 1) + n + 1 + (1 if keep else 0)
+        narrow = sum(1 for t in (a, b, za, f, zf, y1, y2) if t is not None)
+        lib.annotate(bytes=rows * hidden * (4 * streams + a.element_size() * narrow))
+    _depth_join[a.dtype](_ptr(x), _ptr(x_next), _ptr(first), _ptr(kept),
+                         kept.stride(0) if kept is not None else 0, _ptr(depth), n, 1 if keep else 0, float(mult), _ptr(a),
+                         _ptr(bias_a), _ptr(b), _ptr(gain_a), _ptr(gain_b), float(eps), float(weight), _ptr(za), _ptr(ba),
+                         _ptr(f), _ptr(zf), _ptr(bf), *_tanh_norm_args(y1, norm1, hidden, "depth_join"),
+                         *_tanh_norm_args(y2, norm2, hidden, "depth_join"), rows, hidden, _stream())
+
+
 # ------------------------------------------------------------------ rope + cache write
 _rope_kv = _per_dtype("rope_kv", "ek_qk_norm_rope_kv",
                       [_P, c_int, _P, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, c_int,
@@ -343,7 +431,8 @@ def qk_prepare_kv(qkv, n_tokens, q_gain, k_gain, cos, sin, rot_dim, positions, t
     _need_cuda(qkv, cos, sin, positions, token_slot, k_pages, v_pages, block_table, q_bias, k_bias, v_bias)
     check_head_dim(head_dim)
     heads = n_q_heads + (1 if values_from_keys else 2) * n_kv_heads
-    _need(qkv.stride(-1) == 1 and qkv.shape[-1] == heads * head_dim, "qk_prepare_kv: qkv width")
+    _need(qkv.stride(-1) == 1 and (qkv.shape[-1] == heads * head_dim
+                                   or (not write_kv and qkv.shape[-1] == n_q_heads * head_dim)), "qk_prepare_kv: qkv width")
     _need(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous()
           and cos.shape[-1] * 2 == rot_dim, "qk_prepare_kv: 32-bit tables of rot_dim/2 columns")
     _need(k_pages.dtype == qkv.dtype and v_pages.dtype == qkv.dtype, "qk_prepare_kv: cache dtype")
@@ -380,7 +469,7 @@ def qk_prepare_padded_kv(qkv, n_tokens, q_gain, k_gain, cos, sin, rot_dim, posit
     value head is divided by its root mean square over ``value_dim`` values before it is stored."""
     _need_cuda(qkv, cos, sin, positions, token_slot, k_pages, v_pages, block_table, q_bias, k_bias, v_bias)
     check_head_dim(head_dim)
-    heads = n_q_heads + 2 * n_kv_heads
+    heads = n_q_heads + (2 * n_kv_heads if write_kv else 0)      # (keys and values are read only to be stored)
     _need(qkv.stride(-1) == 1 and qkv.shape[-1] >= heads * head_dim, "qk_prepare_padded_kv: row width")
     _need(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous()
           and cos.shape[-1] * 2 == rot_dim, "qk_prepare_padded_kv: 32-bit tables of rot_dim/2 columns")
@@ -406,7 +495,8 @@ def qk_norm_rope_kv(qkv, n_tokens, q_gain, k_gain, cos, sin, rot_dim, positions,
     """In place on the q part of ``qkv`` [T, (NQ + 2 NKV) D]; keys and values go to the pages."""
     _need_cuda(qkv, cos, sin, positions, token_slot, k_pages, v_pages, block_table)
     check_head_dim(head_dim)
-    _need(qkv.stride(-1) == 1 and qkv.shape[-1] == (n_q_heads + 2 * n_kv_heads) * head_dim,
+    _need(qkv.stride(-1) == 1 and (qkv.shape[-1] == (n_q_heads + 2 * n_kv_heads) * head_dim
+                                   or (not write_kv and qkv.shape[-1] == n_q_heads * head_dim)),
           "qk_norm_rope_kv: qkv width")
     _need(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous()
           and cos.shape[-1] * 2 == rot_dim, "qk_norm_rope_kv: 32-bit tables of rot_dim/2 columns")
@@ -456,7 +546,7 @@ def qk_rope_unit_kv(rows, n_tokens, k_col, v_col, cos, sin, rot_dim, positions, 
 # ------------------------------------------------------------------ attention
 _attn_generic = _per_dtype("attention_generic", "ek_attention_generic",
                            [_P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
-                            c_float, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, c_int, _P])
+                            c_float, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, c_int, c_int, c_float, _P])
 _NO_SINK = float("-inf")
 
 
@@ -478,7 +568,7 @@ def _sinks(sinks, n_q_heads):
 def attention_generic(out, q, n_tokens, positions, token_slot, k_pages, v_pages, block_table,
                       n_q_heads, n_kv_heads, head_dim, scale, window=None, n_splits=1,
                       keys_per_split=0, part_acc=None, part_ml=None, sink=None, sinks=None, keep_first=0,
-                      gate=None):
+                      gate=None, chunk=None, softcap=None):
     """out[t, h*D:(h+1)*D] = softmax(scale q.K^T) V over the keys token t may see.  ``sink``: the
     score of one more key without a value that every query sees - exp(sink) is added to the
     softmax denominator (the same in every attention kernel below).  ``sinks`` [NQ] (32-bit):
@@ -489,7 +579,9 @@ def attention_generic(out, q, n_tokens, positions, token_slot, k_pages, v_pages,
     merged from ``part_acc`` [T, NQ, splits, D] / ``part_ml`` [T, NQ, splits, 2] (32-bit).
     ``keep_first`` (with a window): the first ``keep_first`` positions of a sequence stay visible to
     every later token beside its window.  ``gate`` [T, >= NQ] (rows may be a view into wider rows):
-    head h's output at token t is multiplied by sigmoid(gate[t, h]).
+    head h's output at token t is multiplied by sigmoid(gate[t, h]).  ``chunk`` (instead of a window):
+    position p sees only positions of its own chunk, floor(p / chunk).  ``softcap``: a score s becomes
+    softcap * tanh(s / softcap) before the softmax.
     """
     _need_cuda(out, q, positions, token_slot, k_pages, v_pages, block_table, part_acc, part_ml, gate)
     _need(gate is None or (gate.dtype == q.dtype and gate.stride(-1) == 1 and gate.shape[-1] >= n_q_heads),
@@ -502,13 +594,14 @@ def attention_generic(out, q, n_tokens, positions, token_slot, k_pages, v_pages,
         _need(part_acc is not None and part_ml is not None
               and part_acc.numel() >= n_tokens * n_q_heads * n_splits * head_dim
               and part_ml.numel() >= n_tokens * n_q_heads * n_splits * 2, "attention: split buffers")
-    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False)
+    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False, chunk)
     _attn_generic[q.dtype](_ptr(out), _ptr(q), q.stride(0), _ptr(positions), _ptr(token_slot),
                            _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.stride(0),
                            n_tokens, n_q_heads, n_kv_heads, head_dim, float(scale),
                            int(window or 0), n_splits, keys_per_split, _ptr(part_acc),
                            _ptr(part_ml), _sink(sink), _sinks(sinks, n_q_heads), int(keep_first or 0),
-                           _ptr(gate), gate.stride(0) if gate is not None else 0, _stream())
+                           _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk or 0),
+                           float(softcap or 0.0), _stream())
     if n_splits > 1:
         count_extra_launches()               # the merge kernel
 
@@ -564,7 +657,7 @@ def mix_heads(out, parts, mix, positions, n_tokens, n_q_heads, n_kv_heads, head_
 
 _attn_decode_bf16 = Function("attention_decode_bf16", "ek_attention_decode_bf16",
                              [_P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
-                              c_float, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, c_int, _P])
+                              c_float, c_int, c_int, c_int, _P, _P, c_float, _P, c_int, _P, c_int, c_int, c_float, _P])
 
 
 _attn_decode_cross = Function("attention_decode_bf16", "ek_attention_decode_cross_bf16",
@@ -611,9 +704,9 @@ def attention_decode_supported(dtype, head_dim):
 def attention_decode_bf16(out, q, n_tokens, positions, token_slot, k_pages, v_pages, block_table,
                           n_q_heads, n_kv_heads, head_dim, scale, window=None, n_splits=1,
                           keys_per_split=0, part_acc=None, part_ml=None, sink=None, sinks=None, keep_first=0,
-                          gate=None):
+                          gate=None, chunk=None, softcap=None):
     """One query token per row of ``q`` (bfloat16, head_dim a multiple of 32): same contract
-    as :func:`attention_generic` (``keep_first`` and ``gate`` included); ``keys_per_split`` must be a
+    as :func:`attention_generic` (its options included); ``keys_per_split`` must be a
     multiple of 16, or 0 to cut every token's own window into ``n_splits`` equal parts."""
     _need_cuda(out, q, positions, token_slot, k_pages, v_pages, block_table, part_acc, part_ml)
     _need(attention_decode_supported(q.dtype, head_dim),
@@ -626,19 +719,20 @@ def attention_decode_bf16(out, q, n_tokens, positions, token_slot, k_pages, v_pa
         _need(part_acc is not None and part_ml is not None
               and part_acc.numel() >= n_tokens * n_q_heads * n_splits * head_dim
               and part_ml.numel() >= n_tokens * n_q_heads * n_splits * 2, "attention: split buffers")
-    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False)
+    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False, chunk)
     _attn_decode_bf16(_ptr(out), _ptr(q), q.stride(0), _ptr(positions), _ptr(token_slot),
                       _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.stride(0),
                       n_tokens, n_q_heads, n_kv_heads, head_dim, float(scale), int(window or 0),
                       n_splits, keys_per_split, _ptr(part_acc), _ptr(part_ml), _sink(sink),
-                      _sinks(sinks, n_q_heads), int(keep_first or 0), *_gate_args(gate, q, n_q_heads), _stream())
+                      _sinks(sinks, n_q_heads), int(keep_first or 0), *_gate_args(gate, q, n_q_heads),
+                      int(chunk or 0), float(softcap or 0.0), _stream())
     if n_splits > 1:
         count_extra_launches()               # the merge kernel
 
 
 _attn_decode_tma = Function("attention_decode_tma", "ek_attention_decode_tma",
                             [_P, _P, c_int, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int,
-                             c_float, c_int, c_int, _P, c_float, _P])
+                             c_float, c_int, c_int, _P, c_float, c_int, c_float, _P])
 _attn_decode_tma_max = Function("attention_decode_tma", "ek_attention_decode_tma_max_splits", [c_int],
                                 check_status=False)
 DECODE_TMA_PORTABLE_SPLITS = 8
@@ -661,7 +755,8 @@ def attention_decode_tma_supported(dtype, head_dim, n_q_heads, n_kv_heads):
 
 
 def attention_decode_tma(out, q, n_tokens, positions, token_slot, k_pages, v_pages, block_table,
-                         n_q_heads, n_kv_heads, head_dim, scale, window=None, n_splits=1, sink=None):
+                         n_q_heads, n_kv_heads, head_dim, scale, window=None, n_splits=1, sink=None, chunk=None,
+                         softcap=None):
     """One new token per sequence (bfloat16, head size 64 or 128, at most 16 heads a group): the
     cache pages come by TMA, started before the kernel ahead has finished; ``n_splits`` (1 to 8)
     blocks (16 where :func:`decode_tma_max_splits` says so) share a token's pages and merge inside
@@ -683,16 +778,17 @@ def attention_decode_tma(out, q, n_tokens, positions, token_slot, k_pages, v_pag
     _need(1 <= n_splits <= decode_tma_max_splits(head_dim, q.device),
           f"attention_decode_tma: 1 to {decode_tma_max_splits(head_dim, q.device)} splits on this device")
     _need(n_tokens <= 65535, "attention_decode_tma: at most 65535 tokens a call")
-    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False)
+    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, False, chunk)
     _attn_decode_tma(_ptr(out), _ptr(q), q.stride(0), _ptr(positions), _ptr(token_slot),
                      _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table),
                      block_table.stride(0), n_tokens, n_q_heads, n_kv_heads, head_dim, float(scale),
-                     int(window or 0), n_splits, _ptr(tc_status(q.device)), _sink(sink), _stream())
+                     int(window or 0), n_splits, _ptr(tc_status(q.device)), _sink(sink), int(chunk or 0),
+                     float(softcap or 0.0), _stream())
 
 
 _attn_prefill_bf16 = Function("attention_prefill_bf16", "ek_attention_prefill_bf16",
                               [_P, _P, c_int, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int,
-                               c_int, c_int, c_float, c_int, c_float, _P, c_int, _P, c_int, _P])
+                               c_int, c_int, c_float, c_int, c_float, _P, c_int, _P, c_int, c_int, c_float, _P])
 
 
 def attention_prefill_supported(dtype, head_dim, n_q_heads, n_kv_heads):
@@ -702,10 +798,12 @@ def attention_prefill_supported(dtype, head_dim, n_q_heads, n_kv_heads):
 
 def attention_prefill_bf16(out, q, n_tokens, positions, token_slot, cu_seqlens, n_seqs, k_pages,
                            v_pages, block_table, n_q_heads, n_kv_heads, head_dim, scale,
-                           window=None, sink=None, sinks=None, keep_first=0, gate=None):
+                           window=None, sink=None, sinks=None, keep_first=0, gate=None, chunk=None,
+                           softcap=None):
     """Several new tokens per sequence (bfloat16): sequence b owns rows cu_seqlens[b] ..
     cu_seqlens[b+1] of ``q``, which stand at consecutive positions; their keys and values
-    are already in the pages.  ``keep_first`` and ``gate`` as in :func:`attention_generic`."""
+    are already in the pages.  ``keep_first``, ``gate``, ``chunk`` and ``softcap`` as in
+    :func:`attention_generic`."""
     _need_cuda(out, q, positions, token_slot, cu_seqlens, k_pages, v_pages, block_table)
     _need(attention_prefill_supported(q.dtype, head_dim, n_q_heads, n_kv_heads),
           "attention_prefill_bf16: bfloat16, head size a multiple of 16, at most 128 heads a group")
@@ -713,17 +811,18 @@ def attention_prefill_bf16(out, q, n_tokens, positions, token_slot, cu_seqlens, 
     _need(out.is_contiguous() and out.shape[-1] == n_q_heads * head_dim, "attention: out [T, NQ*D]")
     _need(q.stride(-1) == 1 and q.stride(0) % 8 == 0, "attention: dense, 16-byte aligned q rows")
     _need(cu_seqlens.dtype == torch.int32 and cu_seqlens.numel() >= n_seqs + 1, "attention: cu_seqlens")
-    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, True)
+    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, True, chunk)
     _attn_prefill_bf16(_ptr(out), _ptr(q), q.stride(0), _ptr(positions), _ptr(token_slot),
                        _ptr(cu_seqlens), n_seqs, n_tokens, _ptr(k_pages), _ptr(v_pages),
                        _ptr(block_table), block_table.stride(0), n_q_heads, n_kv_heads, head_dim,
                        float(scale), int(window or 0), _sink(sink), _sinks(sinks, n_q_heads),
-                       int(keep_first or 0), *_gate_args(gate, q, n_q_heads), _stream())
+                       int(keep_first or 0), *_gate_args(gate, q, n_q_heads), int(chunk or 0),
+                       float(softcap or 0.0), _stream())
 
 
 _attn_prefill_tc = Function("attention_prefill_tc", "ek_attention_prefill_tc",
                             [_P, _P, c_int, _P, c_int, c_int, _P, _P, c_int, _P, c_int, c_int,
-                             c_int, c_int, c_float, c_int, _P, c_float, _P])
+                             c_int, c_int, c_float, c_int, _P, c_float, c_int, c_float, _P])
 _attn_prefill_tiles = Function("attention_prefill_tc", "ek_attention_prefill_tiles",
                                [_P, c_int, _P, _P, _P, c_int, c_int, c_int, _P])
 _attn_prefill_cross = Function("attention_prefill_bf16", "ek_attention_prefill_cross_bf16",
@@ -793,7 +892,7 @@ def attention_prefill_tiles(tiles, n_tokens, positions, token_slot, cu_seqlens, 
 
 def attention_prefill_tc(out, q, n_tokens, positions, token_slot, cu_seqlens, n_seqs, k_pages,
                          v_pages, block_table, n_q_heads, n_kv_heads, head_dim, scale, window=None,
-                         tiles=None, n_tiles=0, sink=None):
+                         tiles=None, n_tiles=0, sink=None, chunk=None, softcap=None):
     """:func:`attention_prefill_bf16` on tcgen05 tensor cores (head sizes 64 and 128, groups
     that divide 128): TMA-fed pages, scores and P.V in TMEM.  ``tiles`` / ``n_tiles``: the table
     :func:`attention_prefill_tiles` made for this step (made once, before the step's first
@@ -816,18 +915,19 @@ def attention_prefill_tc(out, q, n_tokens, positions, token_slot, cu_seqlens, n_
         torch.cuda.current_stream().synchronize()
     _need(tiles.dtype == torch.int32 and tiles.numel() >= 4 * n_tiles and tiles.data_ptr() % 16 == 0,
           "attention_prefill_tc: the table of tiles")
-    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, True)
+    _attention_cost(q, n_tokens, positions, n_q_heads, n_kv_heads, head_dim, window, True, chunk)
     _attn_prefill_tc(_ptr(out), _ptr(q), q.stride(0), _ptr(tiles), n_tiles, n_tokens, _ptr(k_pages),
                      _ptr(v_pages), k_pages.shape[0], _ptr(block_table), block_table.stride(0), n_q_heads,
                      n_kv_heads, head_dim, float(scale), int(window or 0),
-                     _ptr(tc_status(q.device)), _sink(sink), _stream())
+                     _ptr(tc_status(q.device)), _sink(sink), int(chunk or 0), float(softcap or 0.0), _stream())
 
 
 # ------------------------------------------------------------------ matrix products
 _gemm_f32 = Function("gemm_f32", "ek_gemm_nt_f32",
                      [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P])
 EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_GEGLU = 0, 1, 2, 3      # GEGLU: the gate is the tanh form of GELU
-GATED_EPILOGUES = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU}
+# ("clamped" is EPI_SWIGLU with a gate_limit)
+GATED_EPILOGUES = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_SWIGLU}
 # EPI_BF16 computed by the compiled image that also holds the extended q/k/v epilogue (swapped form):
 # for the other few-row products of a model whose q/k/v product runs there, so that one kernel's code
 # serves them all (see Mixer.product_image)
@@ -880,7 +980,7 @@ def split_scratch(device):
 
 _gemm_tc = Function("gemm_tc_bf16", "ek_gemm_tc_bf16",
                     [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                     _P, _P, c_longlong, c_int, _P, c_int, c_int, c_float, _P, c_int, _P, _P, _P, _P])
+                     _P, _P, c_longlong, c_int, _P, c_int, c_int, c_float, _P, c_int, _P, _P, c_float, _P, _P])
 _tc_status = {}
 TC_SWAP_MAX_ROWS = 64
 
@@ -929,7 +1029,7 @@ def swap_k_split(n_out, k, epilogue):
 
 
 def gemm_tc_bf16(out, x, w, epilogue=EPI_BF16, n_rows=None, swap=None, k_split=None, cluster=True,
-                 row_scale=None, residual=None):
+                 row_scale=None, residual=None, gate_limit=0.0):
     """out = x . w^T (or the SwiGLU of it) on tcgen05 tensor cores with TMA-staged operands.
 
     ``swap`` (default: at most 64 rows) puts the weights on the 128-row side of the MMA and
@@ -940,6 +1040,7 @@ def gemm_tc_bf16(out, x, w, epilogue=EPI_BF16, n_rows=None, swap=None, k_split=N
     Two options of the swapped form carry a norm that was moved out of its own kernel.
     ``row_scale=(ss, size, eps)``: row r of the 32-bit result is multiplied by
     rsqrt(sum(ss[r, :]) / size + eps) before the epilogue (``ss`` [rows, tiles], 32-bit).
+    ``gate_limit`` > 0 (with ``EPI_SWIGLU``): the clamped gate of :func:`act_mul` in place of SiLU.
     ``residual=(stream, gain, ss_out)`` (bfloat16 result, N a multiple of 4): the result is added to
     the 32-bit ``stream`` [rows, N] in place, ``out`` gets stream * gain, and ``ss_out`` [rows,
     ceil(N / 128)] the sum of stream^2 over each 128-column tile.
@@ -991,13 +1092,14 @@ def gemm_tc_bf16(out, x, w, epilogue=EPI_BF16, n_rows=None, swap=None, k_split=N
     _gemm_tc(_ptr(out), _ptr(x), _ptr(w), m, n, k, x.stride(0), w.stride(0), out.stride(0),
              epilogue, 1 if swap else 0, k_split, 1 if cluster else 0, _ptr(partials), _ptr(tickets),
              _SPLIT_PARTIAL_FLOATS, _SPLIT_TICKETS, _ptr(ss_in), ss_tiles, int(size), float(eps),
-             _ptr(stream), ld_stream, _ptr(gain), _ptr(ss_out), _ptr(tc_status(x.device)), _stream())
+             _ptr(stream), ld_stream, _ptr(gain), _ptr(ss_out), float(gate_limit), _ptr(tc_status(x.device)),
+             _stream())
 
 
 _gemm_pair = Function("gemm_pair_bf16", "ek_gemm_pair_bf16",
-                      [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P])
+                      [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
 PAIR_EPI_BF16, PAIR_EPI_ADD_F32, PAIR_EPI_SWIGLU, PAIR_EPI_GEGLU = 0, 1, 2, 4
-PAIR_GATED_EPILOGUES = {"silu": PAIR_EPI_SWIGLU, "gelu_tanh": PAIR_EPI_GEGLU}
+PAIR_GATED_EPILOGUES = {"silu": PAIR_EPI_SWIGLU, "gelu_tanh": PAIR_EPI_GEGLU, "clamped": PAIR_EPI_SWIGLU}
 
 
 def gemm_pair_takes(out, x, w, epilogue) -> bool:
@@ -1008,11 +1110,12 @@ def gemm_pair_takes(out, x, w, epilogue) -> bool:
             and out.stride(0) % (4 if epilogue == PAIR_EPI_ADD_F32 else 8) == 0)
 
 
-def gemm_pair_bf16(out, x, w, epilogue=PAIR_EPI_BF16, n_rows=None):
+def gemm_pair_bf16(out, x, w, epilogue=PAIR_EPI_BF16, n_rows=None, gate_limit=0.0):
     """The product for many rows on pairs of SMs (``tcgen05.mma.cta_group::2``, 256 x 256 tiles, a
     persistent launch).  ``PAIR_EPI_BF16``: out [M, N] = x . w^T in bfloat16; ``PAIR_EPI_ADD_F32``:
     out [M, N] (32-bit) += x . w^T; ``PAIR_EPI_SWIGLU``: out [M, N / 2] = silu(x . wg^T) * (x . wu^T)
-    with w = [gate rows; up rows]; ``PAIR_EPI_GEGLU``: the same with the tanh form of GELU."""
+    with w = [gate rows; up rows]; ``PAIR_EPI_GEGLU``: the same with the tanh form of GELU;
+    ``gate_limit`` > 0 with ``PAIR_EPI_SWIGLU``: the clamped gate of :func:`act_mul`."""
     _need_cuda(out, x, w)
     m = n_rows if n_rows is not None else x.shape[0]
     n, k = w.shape
@@ -1029,7 +1132,7 @@ def gemm_pair_bf16(out, x, w, epilogue=PAIR_EPI_BF16, n_rows=None):
         moved = 2 * (n * k + m * k) + m * n_out * (8 if epilogue == PAIR_EPI_ADD_F32 else 2)
         lib.annotate(bytes=moved, flops=2 * m * n * k, label=f"{n}x{k}")
     _gemm_pair(_ptr(out), _ptr(x), _ptr(w), m, n, k, x.stride(0), w.stride(0), out.stride(0), epilogue,
-               _ptr(tc_status(x.device)), _stream())
+               float(gate_limit), _ptr(tc_status(x.device)), _stream())
 
 
 _gemm_tc_qkv = Function("gemm_tc_bf16", "ek_gemm_tc_qkv_rope",
@@ -1496,7 +1599,7 @@ _xgate_scan = Function("recurrent", "ek_xgate_scan",
                         c_int, c_int, c_int, _P])
 _decay_scan = Function("recurrent", "ek_decay_scan",
                        [_P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_longlong, _P, _P, _P,
-                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P])
+                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P])
 _ssm_out = _per_dtype("recurrent", "ek_ssm_out",
                       [_P, _P, _P, c_int, _P, c_int, c_int, _P, _P, c_float, _P, c_int, c_int, c_int, c_int, _P])
 _xlstm_out = _per_dtype("recurrent", "ek_xlstm_out",
@@ -1634,13 +1737,13 @@ def decay_scan(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot, n_s
     """S_t = a_t S_(t-1) + b_t k_t v_t^T, out_t = S_t^T q_t per head over every sequence's tokens, S
     ([heads, columns, rows] at the start of a slot's state, 32-bit) read and written back.  ``q``, ``k``
     [T, >= kv_heads * dim] (head h reads key head h // (heads / kv_heads)), ``v`` [T, >= heads * vdim],
-    ``a``, ``b`` [T, heads].  ``ones_column``: one more column whose v is 1 (it carries a n + b k and
+    ``a``, ``b`` [T, heads], or [heads] where they are the same for every token.  ``ones_column``: one more column whose v is 1 (it carries a n + b k and
     gives n . q); out is [T, heads * columns]."""
     _need_cuda(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot)
     _need_f32("decay_scan", out, q, k, v, a, b, state)
     cols = vdim + (1 if ones_column else 0)
-    _need(out.shape[-1] == heads * cols and a.is_contiguous() and b.is_contiguous() and a.shape[-1] == heads,
-          "decay_scan: out [T, heads * columns], a and b [T, heads]")
+    _need(out.shape[-1] == heads * cols and a.is_contiguous() and b.is_contiguous() and a.shape[-1] == heads
+          and a.dim() == b.dim(), "decay_scan: out [T, heads * columns], a and b [T, heads] or [heads]")
     _need(state.stride(0) % 4 == 0 and state.shape[-1] >= heads * cols * decay_scan_rows(dim),
           "decay_scan: the state holds S and every slot starts on a 16-byte boundary")
     if lib.recording():
@@ -1649,7 +1752,8 @@ def decay_scan(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot, n_s
                      flops=4 * n_tokens * heads * dim * cols)
     _decay_scan(_ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
                 _ptr(a), _ptr(b), _ptr(state), state.stride(0), _ptr(cu_seqlens), _ptr(positions), _ptr(token_slot),
-                n_seqs, heads, kv_heads, dim, vdim, 1 if ones_column else 0, 1 if write_state else 0, _stream())
+                n_seqs, heads, kv_heads, dim, vdim, 1 if ones_column else 0, 1 if write_state else 0,
+                heads if a.dim() > 1 else 0, _stream())
 
 
 def ssm_out(y, o, x, proj, col_z, d_skip, w, eps, positions, n_tokens, inner, vdim, parts):
@@ -1663,6 +1767,24 @@ def ssm_out(y, o, x, proj, col_z, d_skip, w, eps, positions, n_tokens, inner, vd
         lib.annotate(bytes=n_tokens * inner * (12 + y.element_size()))
     _ssm_out[y.dtype](_ptr(y), _ptr(o), _ptr(x), x.stride(0), _ptr(proj), proj.stride(0), col_z, _ptr(d_skip),
                       _ptr(w), float(eps), _ptr(positions), n_tokens, inner, vdim, parts, _stream())
+
+
+_norm_gate_out = _per_dtype("recurrent", "ek_norm_gate_out",
+                            [_P, _P, _P, c_int, c_int, _P, c_float, _P, c_int, c_int, _P])
+
+
+def norm_gate_out(y, o, proj, col_g, w, eps, positions, n_tokens):
+    """y = o / rms(o) * w * sigmoid(proj[., col_g + c]) in the activation type, the root mean square taken over
+    the whole row (all heads together)."""
+    _need_cuda(y, o, proj, w, positions)
+    _need_f32("norm_gate_out", o, proj, w)
+    inner = y.shape[-1]
+    _need(y.is_contiguous() and o.is_contiguous() and o.shape[-1] == inner == w.numel()
+          and col_g + inner <= proj.shape[-1], "norm_gate_out: y, o, w of one width, the gate within the rows")
+    if lib.recording():
+        lib.annotate(bytes=n_tokens * inner * (8 + y.element_size()))
+    _norm_gate_out[y.dtype](_ptr(y), _ptr(o), _ptr(proj), proj.stride(0), col_g, _ptr(w), float(eps), _ptr(positions),
+                            n_tokens, inner, _stream())
 
 
 def xlstm_out(y, o, m_run, proj, col_g, w, eps, q_scale, positions, n_tokens, heads, vdim):
@@ -1682,10 +1804,12 @@ def xlstm_out(y, o, m_run, proj, col_g, w, eps, q_scale, positions, n_tokens, he
 # ------------------------------------------------------------------ routed experts
 _moe_route = Function("moe", "ek_moe_route", [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P])
 _moe_plan = Function("moe", "ek_moe_plan", [_P, _P, _P, _P, c_int, c_int, _P])
-_moe_up = _per_dtype("moe", "ek_moe_expert_up", [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P])
+_moe_up = _per_dtype("moe", "ek_moe_expert_up",
+                     [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
 _moe_down = _per_dtype("moe", "ek_moe_expert_down", [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P])
-_moe_combine = _per_dtype("moe", "ek_moe_combine", [_P, _P, c_int, c_int, c_int, _P])
-_moe_up_tc = Function("moe", "ek_moe_expert_up_tc", [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P])
+_moe_combine = _per_dtype("moe", "ek_moe_combine", [_P, _P, c_int, c_int, c_int, _P, _P])
+_moe_up_tc = Function("moe", "ek_moe_expert_up_tc",
+                      [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
 _moe_down_tc = Function("moe", "ek_moe_expert_down_tc", [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P])
 
 
@@ -1693,7 +1817,8 @@ def _moe_on_tensor_cores(a, w) -> bool:
     """bfloat16 rows that can be read 16 bytes at a time go to the mma.sync form of the expert products."""
     return (a.dtype == torch.bfloat16 and w.shape[-1] % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 MOE_TILE_ROWS = 64          # must equal kTileRows in csrc/moe.cu
-EXPERT_ACTIVATIONS = {"none": 0, "relu2": 1, "silu": 2, "gelu_tanh": 3}
+EXPERT_ACTIVATIONS = {"none": 0, "relu2": 1, "silu": 2, "gelu_tanh": 3, "clamped": 4}
+ROUTE_WEIGHTS = {"scores_of_chosen": 0, "softmax_of_chosen": 1, "sigmoid": 2}
 
 
 def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
@@ -1701,15 +1826,17 @@ def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
     return -(-n_pairs // MOE_TILE_ROWS) + min(n_experts, n_pairs)
 
 
-def moe_route(sel_expert, sel_weight, logits, n_tokens, n_groups, keep, top, scale, among_chosen=False):
-    """Router: ``logits`` [T, E] 32-bit -> the ``top`` chosen experts and their weights per token.
-    ``among_chosen``: the weights are the softmax over the chosen logits alone (times ``scale``)
-    instead of the chosen scores of the softmax over all experts, divided by their sum."""
+def moe_route(sel_expert, sel_weight, logits, n_tokens, n_groups, keep, top, scale, weights="scores_of_chosen"):
+    """Router: ``logits`` [T, E] 32-bit -> the ``top`` chosen experts and their weights per token, times ``scale``.
+    ``weights``: ``"scores_of_chosen"``, the chosen scores of the softmax over all experts, divided by their sum;
+    ``"softmax_of_chosen"``, the softmax over the chosen logits alone; ``"sigmoid"``, the chosen logits' sigmoids
+    as they are (all groups kept)."""
     _need_cuda(sel_expert, sel_weight, logits)
+    _need(weights in ROUTE_WEIGHTS, f"moe_route: no weights {weights!r}")
     _need(logits.dtype == torch.float32 and logits.is_contiguous() and sel_expert.dtype == torch.int32
           and sel_weight.dtype == torch.float32, "moe_route: 32-bit logits and weights, int32 choices")
     _moe_route(_ptr(sel_expert), _ptr(sel_weight), _ptr(logits), n_tokens, logits.shape[-1], n_groups, keep,
-               top, float(scale), 1 if among_chosen else 0, _stream())
+               top, float(scale), ROUTE_WEIGHTS[weights], _stream())
 
 
 def moe_plan(sorted_pair, tiles, n_tiles, sel_expert, n_pairs, n_experts):
@@ -1717,11 +1844,16 @@ def moe_plan(sorted_pair, tiles, n_tiles, sel_expert, n_pairs, n_experts):
     _moe_plan(_ptr(sorted_pair), _ptr(tiles), _ptr(n_tiles), _ptr(sel_expert), n_pairs, n_experts, _stream())
 
 
-def moe_expert_up(out, x, w, tiles, n_tiles, sorted_pair, n_pairs, top, activation, gated=False):
+def moe_expert_up(out, x, w, tiles, n_tiles, sorted_pair, n_pairs, top, activation, gated=False, limit=0.0,
+                  input_weight=None):
     """out[sorted row] = act(x[token of the pair] . w[expert]^T); ``w`` [E, N, K].  ``gated``: the
     rows of an expert's ``w`` alternate gate, up, gate, up ...; out [pairs, N / 2] holds
-    act(gate) * up, taken from the 32-bit sums."""
-    _need_cuda(out, x, w, tiles, n_tiles, sorted_pair)
+    act(gate) * up, taken from the 32-bit sums (``"clamped"`` as in :func:`act_mul`, with ``limit``).
+    ``input_weight`` [pairs] (32-bit): a pair's input is multiplied by its weight (in the 32-bit sums)."""
+    _need_cuda(out, x, w, tiles, n_tiles, sorted_pair, input_weight)
+    _need(activation != "clamped" or (gated and limit > 0), "moe_expert_up: the clamped gate needs gate rows and a limit")
+    _need(input_weight is None or (input_weight.dtype == torch.float32 and input_weight.is_contiguous()
+                                   and input_weight.numel() >= n_pairs), "moe_expert_up: one 32-bit weight per pair")
     _need(out.dtype == x.dtype == w.dtype and x.is_contiguous() and w.is_contiguous() and out.is_contiguous(),
           "moe_expert_up: one dtype, contiguous")
     e, n, k = w.shape
@@ -1729,11 +1861,13 @@ def moe_expert_up(out, x, w, tiles, n_tiles, sorted_pair, n_pairs, top, activati
         lib.annotate(bytes=x.element_size() * (min(e, n_pairs) * n * k + n_pairs * (n + k)), flops=2 * n_pairs * n * k)
     fn = _moe_up_tc if _moe_on_tensor_cores(x, w) else _moe_up[x.dtype]
     fn(_ptr(out), _ptr(x), _ptr(w), _ptr(tiles), _ptr(n_tiles), _ptr(sorted_pair),
-       moe_max_tiles(n_pairs, e), top, n, k, EXPERT_ACTIVATIONS[activation], 1 if gated else 0, _stream())
+       moe_max_tiles(n_pairs, e), top, n, k, EXPERT_ACTIVATIONS[activation], 1 if gated else 0, float(limit),
+       _ptr(input_weight), _stream())
 
 
 def moe_expert_down(pair_out, a, w, tiles, n_tiles, sorted_pair, pair_weight, n_pairs):
-    """pair_out[pair] = weight[pair] * (a[sorted row] . w[expert]^T) in 32-bit; ``w`` [E, N, K]."""
+    """pair_out[pair] = weight[pair] * (a[sorted row] . w[expert]^T) in 32-bit; ``w`` [E, N, K];
+    ``pair_weight`` None: ones."""
     _need_cuda(pair_out, a, w, tiles, n_tiles, sorted_pair, pair_weight)
     _need(a.dtype == w.dtype and pair_out.dtype == torch.float32 and a.is_contiguous() and w.is_contiguous(),
           "moe_expert_down: 32-bit output")
@@ -1746,12 +1880,15 @@ def moe_expert_down(pair_out, a, w, tiles, n_tiles, sorted_pair, pair_weight, n_
        _ptr(pair_weight), moe_max_tiles(n_pairs, e), n, k, _stream())
 
 
-def moe_combine(out, pair_out, n_tokens, top):
-    _need_cuda(out, pair_out)
+def moe_combine(out, pair_out, n_tokens, top, add=None):
+    """out[t] = sum over the token's ``top`` pairs (+ add[t], in out's type)."""
+    _need_cuda(out, pair_out, add)
     width = out.shape[-1]
+    _need(add is None or (add.dtype == out.dtype and add.is_contiguous() and add.shape[-1] == width),
+          "moe_combine: what is added has out's type and width")
     if lib.recording():
-        lib.annotate(bytes=n_tokens * width * (4 * top + out.element_size()))
-    _moe_combine[out.dtype](_ptr(out), _ptr(pair_out), n_tokens, top, width, _stream())
+        lib.annotate(bytes=n_tokens * width * (4 * top + out.element_size() * (1 if add is None else 2)))
+    _moe_combine[out.dtype](_ptr(out), _ptr(pair_out), n_tokens, top, width, _ptr(add), _stream())
 
 
 def build_all():

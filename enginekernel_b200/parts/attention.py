@@ -16,7 +16,9 @@ load as the reference does (engine/ek_model.py:140-144).
 Optional parameters, all off by default, for designs that differ there:
 
 ``bias``               which of ``"q"``, ``"k"``, ``"v"`` carry a bias (tensors ``q_bias`` ...
-                       [heads * D]); it is added in 32-bit before the head norm.
+                       [heads * D]); it is added in 32-bit before the head norm.  ``"o"``: the output projection
+                       has one (``o_bias`` [H]), added behind its product or, with ``leave_bias=True``, left to the
+                       reader of the result.
 ``values``             ``"keys"``: there is no value projection - a token's value is its key as
                        projected (with bias, before the key's norm and rotation).
 ``query_temperature``  ``(coef, every)``: the query of the token at position p is multiplied by
@@ -36,8 +38,16 @@ Optional parameters, all off by default, for designs that differ there:
                        stored in the cache entry it shares (a run with ``writes_cache=False``).
 ``keep_all_keys``      the cache keeps every key although this layer sees a window (layers that share an
                        entry may see different windows).
-Any of these sends the layer down one path: a single product for everything that reads the input,
-the rotate-and-norm kernel, and the general attention kernel.
+``chunk``              position p sees only its own chunk of positions, floor(p / chunk), counted from the
+                       sequence's first position.
+``cache_window``       how many of a sequence's last keys the cache entry has to keep (default: the window or
+                       the chunk); layers that share an entry name the largest of theirs.
+``softcap``            a score s becomes softcap * tanh(s / softcap) before the softmax.
+``pairing``            ``"neighbours"``: the rotation turns values (2i, 2i + 1) of a head instead of (i, i + rot/2);
+                       the rows of the query and key projections are reordered once at load.
+``value_dim``, ``unit_norm_after_rotation``, ``keep_first`` and ``head_gate`` send the layer down one path: a single
+product for everything that reads the input, a prepare kernel that knows padded heads, and the ``mma.sync`` or the
+general attention kernel.  The others ride on the ordinary path.
 """
 
 from __future__ import annotations
@@ -48,6 +58,7 @@ from ..ops import kernels
 from ..ops.linear import linear, pair_product_wins, row_scale_of, tc_takes
 from ..registry import lookup_part, register_part
 from .base import DeferredNorm, Mixer
+from .rope import neighbours_to_halves
 from .spec import CacheSpec, TensorSpec
 
 FUSE_ROPE_ROWS = 64       # the q/k/v product does norm, rotation and cache write itself up to here
@@ -70,9 +81,13 @@ class Attention(Mixer):
             out.append(TensorSpec(w["gate"], (nh, h)))
         out.append(TensorSpec(w["o"], (h, nh * e)))
         if p.get("qk_norm_eps") is not None:
-            out += [TensorSpec(w["q_norm"], (d,), "gain"), TensorSpec(w["k_norm"], (d,), "gain")]
+            out.append(TensorSpec(w["q_norm"], (d,), "gain"))
+            if p.get("kv_projection", True):     # (else the keys it reads were normed by the run that stored them)
+                out.append(TensorSpec(w["k_norm"], (d,), "gain"))
+        sizes = {"q": nh * d, "k": nkv * d, "v": nkv * e, "o": h}
         for which in p.get("bias") or ():
-            out.append(TensorSpec(w[which + "_bias"], ((nh if which == "q" else nkv) * d,)))
+            if p.get("kv_projection", True) or which in ("q", "o"):
+                out.append(TensorSpec(w[which + "_bias"], (sizes[which],)))
         return out
 
     def __init__(self, spec, dtype, device):
@@ -84,7 +99,19 @@ class Attention(Mixer):
         self.scale = float(self.param("scale"))
         self.qk_norm_eps = spec.params.get("qk_norm_eps")
         self.window = spec.params.get("window")
-        self.biased = tuple(spec.params.get("bias") or ())
+        self.kv_projection = bool(spec.params.get("kv_projection", True))
+        bias = tuple(spec.params.get("bias") or ())
+        self.output_biased = "o" in bias
+        self.biased = tuple(b for b in bias if b != "o" and (self.kv_projection or b == "q"))
+        self.chunk = spec.params.get("chunk")
+        self.softcap = spec.params.get("softcap")
+        self.neighbours = spec.params.get("pairing", "halves") == "neighbours"
+        if spec.params.get("pairing", "halves") not in ("halves", "neighbours"):
+            raise ValueError("attention: pairing is 'halves' or 'neighbours'")
+        if self.chunk is not None and (self.chunk < 1 or self.window or spec.params.get("keep_first")):
+            raise ValueError("attention: a chunk is at least 1 and takes the place of a window")
+        if self.softcap is not None and not self.softcap > 0:
+            raise ValueError("attention: the soft cap must be positive")
         self.values_from_keys = spec.params.get("values", "projection") == "keys"
         self.query_temperature = spec.params.get("query_temperature")
         self.sink = spec.params.get("sink")
@@ -102,17 +129,19 @@ class Attention(Mixer):
         self.unit_norm_eps = spec.params.get("unit_norm_after_rotation")
         self.keep_first = int(spec.params.get("keep_first") or 0)
         self.head_gate = bool(spec.params.get("head_gate"))
-        self.kv_projection = bool(spec.params.get("kv_projection", True))
         self.keep_all_keys = bool(spec.params.get("keep_all_keys")) or self.keep_first > 0
         self.general = (self.value_dim != self.head_dim or self.unit_norm_eps is not None or self.keep_first > 0
-                        or self.head_gate or not self.kv_projection)
+                        or self.head_gate)
+        if not self.kv_projection and self.values_from_keys:
+            raise ValueError("attention: values from keys need a key projection")
         #: the head size the cache and the kernels see
         self.padded_dim = self.head_dim
         if self.general:
-            if not self._plain or self.qk_norm_eps is not None or self.sink is not None:
-                raise ValueError("attention: value_dim, unit_norm_after_rotation, keep_first, head_gate and "
-                                 "kv_projection do not combine with biases, values from keys, a query "
-                                 "temperature, the gained q/k norm or a sink")
+            if self.values_from_keys or self.query_temperature is not None or self.sink is not None:
+                raise ValueError("attention: value_dim, unit_norm_after_rotation, keep_first and head_gate do not "
+                                 "combine with values from keys, a query temperature or a sink")
+            if self.unit_norm_eps is not None and (self.biased or self.qk_norm_eps is not None):
+                raise ValueError("attention: unit_norm_after_rotation does not combine with biases or the gained norm")
             if self.keep_first and not self.window:
                 raise ValueError("attention: keep_first needs a window")
             # (a multiple of 32 where the 16-bit attention kernels can take it: at most a quarter more)
@@ -123,13 +152,19 @@ class Attention(Mixer):
             kernels.check_head_dim(self.padded_dim)
             # (this path takes normalised activations and returns a plain tensor)
             self.takes_deferred_norm = self.defers_norm = False
+        if self.output_biased:                   # (the product alone is not the result yet)
+            self.defers_norm = False
         pos = spec.params.get("position")
         self.position = lookup_part("position", pos.kind)(pos, dtype, device) if pos else None
+        if self.neighbours and self.position is not None and \
+                int(getattr(self.position, "rotary_dim", 0)) > self.head_dim:
+            raise ValueError("attention: the rotation covers more values than a head has")
         self.w_qkv = self.w_o = self.q_gain = self.k_gain = None
 
     def cache_spec(self):
+        window = self.spec.params.get("cache_window") or self.window or self.chunk
         return CacheSpec("kv", heads=self.num_kv_heads, head_dim=self.padded_dim,
-                         window=None if self.keep_all_keys else self.window)
+                         window=None if self.keep_all_keys else window)
 
     def prepare(self, max_positions):
         if self.position is not None:
@@ -154,23 +189,41 @@ class Attention(Mixer):
                                             ctx.n_seqs, self.num_heads, self.num_kv_heads, self.head_dim)
         ctx.shared[key] = (tiles, n)
 
+    def _by_head(self, t, n, reorder):
+        """[n * size, ...] -> [n * padded_dim, ...]: a head's values in the kernels' order (``reorder``: they turn
+        with the rotation), zeros behind them."""
+        size = t.shape[0] // n
+        t = t.reshape(n, size, *t.shape[1:])
+        if reorder and self.neighbours and self.position is not None:
+            t = t.index_select(1, neighbours_to_halves(size, int(self.position.rotary_dim)).to(t.device))
+        if size != self.padded_dim:
+            out = torch.zeros((n, self.padded_dim) + tuple(t.shape[2:]), dtype=t.dtype, device=t.device)
+            out[:, :size] = t
+            t = out
+        return t.reshape(n * self.padded_dim, *t.shape[2:])
+
+    def _load_vectors(self, tensors):
+        """Biases of the projections and gains of the head norms, in 32-bit and in the kernels' order."""
+        w, f32 = self.spec.weights, torch.float32
+        for which in self.biased:
+            n = self.num_heads if which == "q" else self.num_kv_heads
+            self.bias[which] = self._by_head(tensors[w[which + "_bias"]].to(f32), n, which != "v").contiguous()
+        if self.qk_norm_eps is not None:
+            self.q_gain = self._by_head(tensors[w["q_norm"]].to(f32), 1, True).contiguous()
+            if self.kv_projection:
+                self.k_gain = self._by_head(tensors[w["k_norm"]].to(f32), 1, True).contiguous()
+        if self.output_biased:
+            self.output_bias = tensors[w["o_bias"]].to(f32).contiguous()
+
     def _load_general(self, tensors):
         """[q | k | v | gate] as one weight, every head padded with zero rows to ``padded_dim``, zero rows
         up to a multiple of 64; ``o`` with zero columns where the value heads are padded."""
         w, big = self.spec.weights, self.padded_dim
-
-        def heads(t, n, size):
-            t = t.view(n, size, self.hidden)
-            if size == big:
-                return t.reshape(n * big, self.hidden)
-            out = torch.zeros((n, big, self.hidden), dtype=t.dtype, device=t.device)
-            out[:, :size] = t
-            return out.view(n * big, self.hidden)
-
-        rows = [heads(tensors[w["q"]], self.num_heads, self.head_dim)]
+        self._load_vectors(tensors)
+        rows = [self._by_head(tensors[w["q"]], self.num_heads, True)]
         if self.kv_projection:
-            rows += [heads(tensors[w["k"]], self.num_kv_heads, self.head_dim),
-                     heads(tensors[w["v"]], self.num_kv_heads, self.value_dim)]
+            rows += [self._by_head(tensors[w["k"]], self.num_kv_heads, True),
+                     self._by_head(tensors[w["v"]], self.num_kv_heads, False)]
         if self.head_gate:
             rows.append(tensors[w["gate"]])
         n = sum(r.shape[0] for r in rows)
@@ -184,26 +237,36 @@ class Attention(Mixer):
             o = wide
         self.w_o = o.reshape(self.hidden, self.num_heads * big).to(self.dtype).contiguous()
 
-    def _forward_general(self, x, ctx, entry, writes_cache):
+    def _forward_general(self, x, ctx, entry, writes_cache, leave_bias=False):
         t, big, nh, nkv = ctx.n_tokens, self.padded_dim, self.num_heads, self.num_kv_heads
         pos = self.position
         rows = linear(x, self.w_qkv, ctx, "qkv", n_rows=t)
         k_col = nh * big
         gate_col = k_col + (2 * nkv * big if self.kv_projection else 0)
-        kernels.qk_rope_unit_kv(
-            rows, t, k_col, k_col + nkv * big, pos.cos if pos else _no_table(self.device),
-            pos.sin if pos else _no_table(self.device), pos.rotary_dim if pos else 0, ctx.positions,
-            ctx.token_slot, entry.k_pages, entry.v_pages, entry.block_table, nh, nkv, big, self.head_dim,
-            self.unit_norm_eps or 0.0, unit=self.unit_norm_eps is not None,
-            write_kv=writes_cache and self.kv_projection)
+        if self.qk_norm_eps is not None or self.biased:
+            kernels.qk_prepare_padded_kv(
+                rows, t, self.q_gain, self.k_gain, pos.cos if pos else _no_table(self.device),
+                pos.sin if pos else _no_table(self.device), pos.rotary_dim if pos else 0, ctx.positions,
+                ctx.token_slot, entry.k_pages, entry.v_pages, entry.block_table, nh, nkv, big,
+                self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, self.head_dim,
+                write_kv=writes_cache and self.kv_projection, q_bias=self.bias["q"], k_bias=self.bias["k"],
+                v_bias=self.bias["v"])
+        else:
+            kernels.qk_rope_unit_kv(
+                rows, t, k_col, k_col + nkv * big, pos.cos if pos else _no_table(self.device),
+                pos.sin if pos else _no_table(self.device), pos.rotary_dim if pos else 0, ctx.positions,
+                ctx.token_slot, entry.k_pages, entry.v_pages, entry.block_table, nh, nkv, big, self.head_dim,
+                self.unit_norm_eps or 0.0, unit=self.unit_norm_eps is not None,
+                write_kv=writes_cache and self.kv_projection)
         out = ctx.workspace.get("attn_out", (t, nh * big), self.dtype)
-        visible = min(ctx.max_context, self.window + self.keep_first) if self.window else ctx.max_context
+        visible = self._visible(ctx)
         gate = rows[:, gate_col:] if self.head_gate else None
+        mask = {"chunk": self.chunk, "softcap": self.softcap}
         if not ctx.is_decode and kernels.attention_prefill_supported(self.dtype, big, nh, nkv):
             kernels.attention_prefill_bf16(out, rows, t, ctx.positions, ctx.token_slot, ctx.cu_seqlens, ctx.n_seqs,
                                            entry.k_pages, entry.v_pages, entry.block_table, nh, nkv, big, self.scale,
-                                           self.window, keep_first=self.keep_first, gate=gate)
-            return linear(out, self.w_o, ctx, "attn_proj", n_rows=t)
+                                           self.window, keep_first=self.keep_first, gate=gate, **mask)
+            return self._project(out, ctx, None, leave_bias)
         if ctx.is_decode and kernels.attention_decode_supported(self.dtype, big):
             # blocks = tokens x KV heads (x 16-row blocks of the group), three fit an SM: every token's own
             # window is cut so that the blocks about fill the machine, never finer than two pages a split
@@ -215,8 +278,8 @@ class Attention(Mixer):
                 ml = ctx.workspace.get("attn_part_ml", (t, nh, splits, 2), torch.float32)
             kernels.attention_decode_bf16(out, rows, t, ctx.positions, ctx.token_slot, entry.k_pages, entry.v_pages,
                                           entry.block_table, nh, nkv, big, self.scale, self.window, splits, 0, acc, ml,
-                                          keep_first=self.keep_first, gate=gate)
-            return linear(out, self.w_o, ctx, "attn_proj", n_rows=t)
+                                          keep_first=self.keep_first, gate=gate, **mask)
+            return self._project(out, ctx, None, leave_bias)
         splits, per_split, acc, ml = 1, 0, None, None
         blocks = t * nh
         if blocks < 2 * kernels.sm_count(self.device) and visible > 512:
@@ -229,37 +292,53 @@ class Attention(Mixer):
             ml = ctx.workspace.get("attn_part_ml", (t, nh, splits, 2), torch.float32)
         kernels.attention_generic(out, rows, t, ctx.positions, ctx.token_slot, entry.k_pages, entry.v_pages,
                                   entry.block_table, nh, nkv, big, self.scale, self.window, splits, per_split,
-                                  acc, ml, keep_first=self.keep_first, gate=gate)
-        return linear(out, self.w_o, ctx, "attn_proj", n_rows=t)
+                                  acc, ml, keep_first=self.keep_first, gate=gate, **mask)
+        return self._project(out, ctx, None, leave_bias)
 
     def load(self, tensors):
         if self.general:
             return self._load_general(tensors)
         w = self.spec.weights
-        rows = [tensors[w["q"]], tensors[w["k"]]] + ([] if self.values_from_keys else [tensors[w["v"]]])
+        self._load_vectors(tensors)
+        rows = [self._by_head(tensors[w["q"]], self.num_heads, True)]
+        if self.kv_projection:
+            rows.append(self._by_head(tensors[w["k"]], self.num_kv_heads, True))
+            if not self.values_from_keys:
+                rows.append(tensors[w["v"]])
         self.w_qkv = torch.cat(rows, dim=0).to(self.dtype).contiguous()
-        for which in self.biased:
-            self.bias[which] = tensors[w[which + "_bias"]].to(torch.float32).contiguous()
         self.w_o = tensors[w["o"]].to(self.dtype).contiguous()
-        if self.qk_norm_eps is not None:
-            self.q_gain = tensors[w["q_norm"]].to(torch.float32).contiguous()
-            self.k_gain = tensors[w["k_norm"]].to(torch.float32).contiguous()
 
     def bytes_read_per_step(self, n_tokens):
         return sum(t.numel() * t.element_size() for t in (self.w_qkv, self.w_o, self.q_gain, self.k_gain,
-                                                          *self.bias.values()) if t is not None)
+                                                          self.output_bias, *self.bias.values()) if t is not None)
 
     # ------------------------------------------------------------------
     takes_deferred_norm = True
     defers_norm = True
 
-    def forward(self, x, ctx, entry, writes_cache=True, defer=None):
+    def _visible(self, ctx):
+        """Keys a token of this step sees at most."""
+        if self.chunk:
+            return min(ctx.max_context, self.chunk)
+        return min(ctx.max_context, self.window + self.keep_first) if self.window else ctx.max_context
+
+    def _project(self, out, ctx, defer, leave_bias):
+        y = linear(out, self.w_o, ctx, "attn_proj", n_rows=ctx.n_tokens, defer=None if self.output_biased else defer,
+                   image=self.product_image())
+        if self.output_bias is None or leave_bias:
+            return y
+        biased = ctx.workspace.get("attn_proj_biased", (ctx.n_tokens, self.hidden), self.dtype)
+        kernels.bias_act(biased, y, self.output_bias, None, n_rows=ctx.n_tokens)
+        return biased
+
+    def forward(self, x, ctx, entry, writes_cache=True, defer=None, leave_bias=False):
         t = ctx.n_tokens
         pos = self.position
         if self.general:
             if isinstance(x, DeferredNorm):
                 raise kernels.KernelError("this attention layer takes normalised activations, not a deferred norm")
-            return self._forward_general(x, ctx, entry, writes_cache)
+            return self._forward_general(x, ctx, entry, writes_cache, leave_bias)
+        writes_cache = writes_cache and self.kv_projection
         if self._fuses_rope(x, ctx):
             # few rows, heads of 128: norm, rotation and cache write ride on the product's epilogue
             row_scale, xin = (row_scale_of(x), x.scaled) if isinstance(x, DeferredNorm) else (None, x)
@@ -271,7 +350,7 @@ class Attention(Mixer):
                 self.num_heads, self.num_kv_heads, write_kv=writes_cache, row_scale=row_scale)
             out = ctx.workspace.get("attn_out", (t, self.num_heads * self.head_dim), self.dtype)
             self._attend(out, qkv, ctx, entry)
-            return linear(out, self.w_o, ctx, "attn_proj", n_rows=t, defer=defer, image=self.product_image())
+            return self._project(out, ctx, defer, leave_bias)
         if self._fuses_prepare(x, ctx):
             # the same for designs with biases, a query temperature, values taken from the keys,
             # or no rotation at all
@@ -287,7 +366,7 @@ class Attention(Mixer):
                 q_temperature=self.query_temperature, values_from_keys=self.values_from_keys)
             out = ctx.workspace.get("attn_out", (t, self.num_heads * self.head_dim), self.dtype)
             self._attend(out, qkv, ctx, entry)
-            return linear(out, self.w_o, ctx, "attn_proj", n_rows=t, defer=defer, image=self.product_image())
+            return self._project(out, ctx, defer, leave_bias)
         if self._fuses_rope_of_many_rows(x, ctx):
             # many rows, heads of 128: the same on the epilogue of the product on pairs of SMs
             qkv = ctx.workspace.get("qkv", (t, self.w_qkv.shape[0]), self.dtype)
@@ -298,7 +377,7 @@ class Attention(Mixer):
                 self.num_heads, self.num_kv_heads, write_kv=writes_cache)
             out = ctx.workspace.get("attn_out", (t, self.num_heads * self.head_dim), self.dtype)
             self._attend(out, qkv, ctx, entry)
-            return linear(out, self.w_o, ctx, "attn_proj", n_rows=t, defer=defer, image=self.product_image())
+            return self._project(out, ctx, defer, leave_bias)
         qkv = linear(x, self.w_qkv, ctx, "qkv", n_rows=t)
         prepare = (qkv, t, self.q_gain, self.k_gain,
                    pos.cos if pos else _no_table(self.device), pos.sin if pos else _no_table(self.device),
@@ -314,7 +393,7 @@ class Attention(Mixer):
                                   values_from_keys=self.values_from_keys)
         out = ctx.workspace.get("attn_out", (t, self.num_heads * self.head_dim), self.dtype)
         self._attend(out, qkv, ctx, entry)
-        return linear(out, self.w_o, ctx, "attn_proj", n_rows=t, defer=defer, image=self.product_image())
+        return self._project(out, ctx, defer, leave_bias)
 
     @property
     def _plain(self):
@@ -325,7 +404,7 @@ class Attention(Mixer):
     def _fuses_rope(self, x, ctx):
         xin = x.scaled if isinstance(x, DeferredNorm) else x
         pos = self.position
-        return (self._plain and self.dtype == torch.bfloat16 and ctx.n_tokens <= FUSE_ROPE_ROWS
+        return (self._plain and self.kv_projection and self.dtype == torch.bfloat16 and ctx.n_tokens <= FUSE_ROPE_ROWS
                 and self.head_dim == kernels.QKV_ROPE_HEAD_DIM and pos is not None
                 and getattr(pos, "rotary_dim", 0) == self.head_dim and tc_takes(xin, self.w_qkv))
 
@@ -340,12 +419,12 @@ class Attention(Mixer):
 
     def _fuses_prepare(self, x, ctx):
         xin = x.scaled if isinstance(x, DeferredNorm) else x
-        return (self.product_image() == "extended" and ctx.n_tokens <= FUSE_ROPE_ROWS
+        return (self.product_image() == "extended" and self.kv_projection and ctx.n_tokens <= FUSE_ROPE_ROWS
                 and tc_takes(xin, self.w_qkv))
 
     def _fuses_rope_of_many_rows(self, x, ctx):
         pos = self.position
-        if (not self._plain or isinstance(x, DeferredNorm) or self.dtype != torch.bfloat16
+        if (not self._plain or not self.kv_projection or isinstance(x, DeferredNorm) or self.dtype != torch.bfloat16
                 or self.head_dim != kernels.QKV_ROPE_HEAD_DIM or pos is None
                 or getattr(pos, "rotary_dim", 0) != self.head_dim):
             return False
@@ -354,7 +433,8 @@ class Attention(Mixer):
 
     def _attend(self, out, qkv, ctx, entry):
         t = ctx.n_tokens
-        visible = min(ctx.max_context, self.window) if self.window else ctx.max_context
+        visible = self._visible(ctx)
+        mask = {"chunk": self.chunk, "softcap": self.softcap}
         fast_decode = ctx.is_decode and kernels.attention_decode_supported(self.dtype, self.head_dim)
         if not ctx.is_decode and kernels.attention_prefill_supported(
                 self.dtype, self.head_dim, self.num_heads, self.num_kv_heads):
@@ -371,7 +451,7 @@ class Attention(Mixer):
             prefill(
                 out, qkv, t, ctx.positions, ctx.token_slot, ctx.cu_seqlens, ctx.n_seqs,
                 entry.k_pages, entry.v_pages, entry.block_table, self.num_heads, self.num_kv_heads,
-                self.head_dim, self.scale, self.window, sink=self.sink, **extra)
+                self.head_dim, self.scale, self.window, sink=self.sink, **mask, **extra)
             return
         if ctx.is_decode and t <= 65535 and kernels.attention_decode_tma_supported(
                 self.dtype, self.head_dim, self.num_heads, self.num_kv_heads):
@@ -387,7 +467,7 @@ class Attention(Mixer):
             kernels.attention_decode_tma(
                 out, qkv, t, ctx.positions, ctx.token_slot, entry.k_pages, entry.v_pages,
                 entry.block_table, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
-                self.window, splits, sink=self.sink)
+                self.window, splits, sink=self.sink, **mask)
             return
         if fast_decode:
             # blocks = tokens x KV heads (x 16-row blocks of the group); three fit an SM.  Split
@@ -403,7 +483,7 @@ class Attention(Mixer):
         else:
             blocks = t * self.num_heads
             splits = 1
-            if blocks < 2 * kernels.sm_count(self.device) and ctx.max_context > 512:
+            if blocks < 2 * kernels.sm_count(self.device) and visible > 512:
                 splits = max(1, min(-(-visible // 256), -(-4 * kernels.sm_count(self.device) // blocks), 64))
             unit = 128
         per_split, acc, ml = 0, None, None
@@ -418,7 +498,7 @@ class Attention(Mixer):
                 entry.block_table, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
                 self.window, splits, per_split, acc, ml)
         fn = kernels.attention_decode_bf16 if fast_decode else kernels.attention_generic
-        fn(*args, sink=self.sink)
+        fn(*args, sink=self.sink, **mask)
 
 
 _EMPTY = {}

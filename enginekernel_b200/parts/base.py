@@ -118,6 +118,17 @@ class WeightedPair:
         self.a, self.weight_a, self.b, self.weight_b = a, float(weight_a), b, float(weight_b)
 
 
+class NormedPair:
+    """The same for two mixers whose results are normed over their width before they are summed:
+    weight * (a / rms(a) * gain_a + b / rms(b) * gain_b), the root mean squares with ``eps`` inside the root,
+    the gains 32-bit vectors."""
+    __slots__ = ("a", "gain_a", "b", "gain_b", "eps", "weight")
+
+    def __init__(self, a, gain_a, b, gain_b, eps, weight):
+        self.a, self.gain_a, self.b, self.gain_b = a, gain_a, b, gain_b
+        self.eps, self.weight = float(eps), float(weight)
+
+
 class Part:
     """Base of all parts."""
     role = ""
@@ -156,6 +167,11 @@ class Norm(Part):
         the whole stream row and so can be a :class:`DeferredNorm`; else None."""
         return None
 
+    def pointwise(self):
+        """(alpha [1], weight [size], shift [size] in 32-bit) if this norm is tanh(alpha * x) * weight + shift,
+        element by element, and so can ride in a kernel that writes the stream; else None."""
+        return None
+
     def forward(self, stream, ctx: StepContext, add=None, rows=None, n_rows=None,
                 write_back=True):
         raise NotImplementedError
@@ -177,6 +193,8 @@ class Mixer(Part):
     #: ``forward`` takes a DeferredNorm for ``x`` / takes ``defer=(stream, norm)`` and may return one
     takes_deferred_norm = False
     defers_norm = False
+    #: a bias of the result that ``forward(..., leave_bias=True)`` leaves to whoever reads it (32-bit, or None)
+    output_bias = None
 
     def cache_spec(self) -> Optional[CacheSpec]:
         """What one cache entry of this mixer holds per sequence (None: nothing)."""

@@ -35,15 +35,8 @@ from ..ops.linear import linear
 from ..registry import lookup_part, register_part
 from .attention import _no_table
 from .base import Mixer
+from .rope import neighbours_to_halves
 from .spec import CacheSpec, TensorSpec
-
-
-def neighbours_to_halves(dim: int, rotary_dim: int) -> torch.Tensor:
-    """Order of a head's values that turns the pairs (2i, 2i + 1) of its first ``rotary_dim`` values into
-    the pairs (i, i + rotary_dim / 2): new[i] = old[order[i]]."""
-    even = list(range(0, rotary_dim, 2))
-    odd = list(range(1, rotary_dim, 2))
-    return torch.tensor(even + odd + list(range(rotary_dim, dim)), dtype=torch.long)
 
 
 @register_part("mixer", "mixed_head_attention")

@@ -1,9 +1,11 @@
 """Gated feed-forward: down(act(gate(x)) * up(x)), no biases; act is SiLU (SwiGLU) or the
-tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
+tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); or, ``"clamped"`` with a ``limit``,
+down(g sigmoid(1.702 g) (u + 1)) with g = min(gate(x), limit) and u = clamp(up(x), -limit, limit).
 
 engine/ek_model.py:205-209 with engine/ek_kernels.py:125-143; gate and up are
 concatenated at load (gate rows first, engine/ek_model.py:145-147).  Parameters:
-``hidden_size``, ``intermediate_size``, ``activation`` ("silu", the default, or "gelu_tanh").  Tensors: ``gate``,
+``hidden_size``, ``intermediate_size``, ``activation`` ("silu", the default, "gelu_tanh" or "clamped"),
+``limit`` (with "clamped").  ``name`` (default "mlp") names the scratch buffers, for a layer that runs two.  Tensors: ``gate``,
 ``up`` [I, H], ``down`` [H, I].
 """
 
@@ -35,6 +37,10 @@ class GatedMLP(FeedForward):
         if self.activation not in kernels.GATE_ACTIVATIONS:
             raise ValueError(f"gated_mlp has no activation {self.activation!r} "
                              f"({', '.join(kernels.GATE_ACTIVATIONS)})")
+        self.limit = float(spec.params.get("limit") or 0.0)
+        if self.activation == "clamped" and not self.limit > 0:
+            raise ValueError("gated_mlp: the clamped gate needs a positive limit")
+        self.name = spec.params.get("name", "mlp")
         self.w_gate_up = self.w_down = None
 
     def load(self, tensors):
@@ -56,24 +62,24 @@ class GatedMLP(FeedForward):
             row_scale, x = row_scale_of(x), x.scaled
         if self.dtype == torch.bfloat16 and t <= kernels.TC_SWAP_MAX_ROWS and tc_takes(x, self.w_gate_up):
             # gate and up rows share a tile, so act(gate) * up is formed in the epilogue
-            act = ctx.workspace.get("mlp_act", (t, self.inter), self.dtype)
+            act = ctx.workspace.get(self.name + "_act", (t, self.inter), self.dtype)
             kernels.gemm_tc_bf16(act, x, self.w_gate_up, kernels.GATED_EPILOGUES[self.activation], n_rows=t,
-                                 swap=True, row_scale=row_scale)
+                                 swap=True, row_scale=row_scale, gate_limit=self.limit)
         elif row_scale is not None:
             raise kernels.KernelError("a deferred norm reached a product that cannot scale its rows")
         elif self.dtype == torch.bfloat16 and pair_product_wins(
-                ctx.workspace.get("mlp_act", (t, self.inter), self.dtype), x, self.w_gate_up, t,
+                ctx.workspace.get(self.name + "_act", (t, self.inter), self.dtype), x, self.w_gate_up, t,
                 kernels.PAIR_GATED_EPILOGUES[self.activation]):
             # many rows: the pair of blocks that shares a tile stages gate rows in one block and the
             # matching up rows in the other, and the epilogue forms act(gate) * up from the 32-bit sums
-            act = ctx.workspace.get("mlp_act", (t, self.inter), self.dtype)
+            act = ctx.workspace.get(self.name + "_act", (t, self.inter), self.dtype)
             kernels.gemm_pair_bf16(act, x, self.w_gate_up, kernels.PAIR_GATED_EPILOGUES[self.activation],
-                                   n_rows=t)
+                                   n_rows=t, gate_limit=self.limit)
         else:
-            gu = linear(x, self.w_gate_up, ctx, "mlp_gate_up", n_rows=t)
-            act = ctx.workspace.get("mlp_act", (t, self.inter), self.dtype)
-            kernels.act_mul(act, gu, self.activation, n_rows=t)
-        return linear(act, self.w_down, ctx, "mlp_down", n_rows=t, defer=defer, image=self.product_image)
+            gu = linear(x, self.w_gate_up, ctx, self.name + "_gate_up", n_rows=t)
+            act = ctx.workspace.get(self.name + "_act", (t, self.inter), self.dtype)
+            kernels.act_mul(act, gu, self.activation, n_rows=t, limit=self.limit)
+        return linear(act, self.w_down, ctx, self.name + "_down", n_rows=t, defer=defer, image=self.product_image)
 
 
 @register_part("feed_forward", "dense_mlp")

@@ -11,14 +11,20 @@ weights are the softmax over those chosen logits alone, times ``scale``.  With `
 W_down,e (act(W_gate,e h) * (W_up,e h)) (tensors ``gate_<e>`` [I, hidden] beside ``up_<e>``; gate and up rows
 are interleaved at load, so that one product gives both and its epilogue their 32-bit product).
 
+With ``weights="sigmoid"`` the scores are the logits' sigmoids, each for itself, and the weights are the chosen scores
+times ``scale``, not divided by their sum.  With ``weigh="input"`` the weight multiplies the expert's input instead of
+its output: out = sum over the chosen experts of W_down,e act(W_up,e (weight h)); the product is linear, so the
+weight joins it in the 32-bit sums.  ``shared``, a feed-forward PartSpec, runs for every token and is added.
+
 Experts have no biases; ``activation`` is ``"relu2"`` (the square of relu), ``"silu"``,
-``"gelu_tanh"`` or ``"none"``.  The choice is made and used on the device: a kernel sorts the (token,
+``"gelu_tanh"``, ``"none"`` or, for gated experts, ``"clamped"`` with a ``limit`` (``parts/mlp.py``).  The choice is made and used on the device: a kernel sorts the (token,
 choice) pairs by expert and cuts every expert's stretch into row tiles, and the two expert products
 walk those tiles, so nothing here waits for the device and the step can be captured in a graph.
 
 Parameters: ``hidden_size``, ``intermediate_size`` (of one expert), ``experts``, ``top``, ``groups``
 (default 1), ``keep`` (default: all groups), ``scale``, ``activation``, ``gated`` (default False), ``weights``
-(``"scores_of_chosen"``, the default, or ``"softmax_of_chosen"``).  Tensors: ``router`` [E, hidden]
+(``"scores_of_chosen"``, the default, ``"softmax_of_chosen"`` or ``"sigmoid"``), ``weigh`` (``"output"``, the default, or
+``"input"``), ``limit``, ``shared``.  Tensors: ``router`` [E, hidden]
 and per expert ``up_<e>`` [I, hidden], ``down_<e>`` [hidden, I].
 """
 
@@ -28,7 +34,7 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import linear
-from ..registry import register_part
+from ..registry import lookup_part, register_part
 from .base import FeedForward
 from .spec import TensorSpec
 
@@ -44,6 +50,9 @@ class RoutedExperts(FeedForward):
             if p.get("gated"):
                 out.append(TensorSpec(w[f"gate_{e}"], (i, h)))
             out += [TensorSpec(w[f"up_{e}"], (i, h)), TensorSpec(w[f"down_{e}"], (h, i))]
+        shared = p.get("shared")
+        if shared is not None:
+            out += lookup_part("feed_forward", shared.kind).tensors(shared)
         return out
 
     def __init__(self, spec, dtype, device):
@@ -56,7 +65,15 @@ class RoutedExperts(FeedForward):
         self.activation = spec.params.get("activation", "relu2")
         self.gated = bool(spec.params.get("gated"))
         self.weights = spec.params.get("weights", "scores_of_chosen")
-        if self.weights not in ("scores_of_chosen", "softmax_of_chosen"):
+        self.weigh_input = spec.params.get("weigh", "output") == "input"
+        self.limit = float(spec.params.get("limit") or 0.0)
+        shared = spec.params.get("shared")
+        self.shared = None if shared is None else lookup_part("feed_forward", shared.kind)(shared, dtype, device)
+        if spec.params.get("weigh", "output") not in ("output", "input"):
+            raise ValueError("routed_experts: the weight joins the expert's input or its output")
+        if self.activation == "clamped" and not (self.gated and self.limit > 0):
+            raise ValueError("routed_experts: the clamped gate needs gated experts and a positive limit")
+        if self.weights not in kernels.ROUTE_WEIGHTS:
             raise ValueError(f"routed_experts has no weights {self.weights!r}")
         if self.activation not in kernels.EXPERT_ACTIVATIONS:
             raise ValueError(f"routed_experts has no activation {self.activation!r}")
@@ -68,6 +85,8 @@ class RoutedExperts(FeedForward):
 
     def load(self, tensors):
         w = self.spec.weights
+        if self.shared is not None:
+            self.shared.load(tensors)
         self.w_router = tensors[w["router"]].to(self.dtype).contiguous()
         ups = [tensors[w[f"up_{e}"]] for e in range(self.experts)]
         if self.gated:               # rows gate_0, up_0, gate_1, up_1, ... of every expert
@@ -80,7 +99,8 @@ class RoutedExperts(FeedForward):
         """The router and the experts that ``n_tokens`` tokens can reach at most."""
         touched = min(self.experts, n_tokens * self.top)
         per_expert = (self.w_up[0].numel() + self.w_down[0].numel()) * self.w_up.element_size()
-        return self.w_router.numel() * self.w_router.element_size() + touched * per_expert
+        shared = self.shared.bytes_read_per_step(n_tokens) if self.shared is not None else 0
+        return self.w_router.numel() * self.w_router.element_size() + touched * per_expert + shared
 
     def forward(self, x, ctx):
         t, ws, top = ctx.n_tokens, ctx.workspace, self.top
@@ -89,16 +109,21 @@ class RoutedExperts(FeedForward):
         chosen = ws.get("moe_chosen", (t, top), torch.int32)
         weight = ws.get("moe_weight", (t, top), torch.float32)
         kernels.moe_route(chosen, weight, logits, t, self.groups, self.keep, top, self.scale,
-                          among_chosen=self.weights == "softmax_of_chosen")
+                          weights=self.weights)
         sorted_pair = ws.get("moe_sorted", (pairs,), torch.int32)
         tiles = ws.get("moe_tiles", (kernels.moe_max_tiles(pairs, self.experts), 3), torch.int32)
         n_tiles = ws.get("moe_n_tiles", (1,), torch.int32)
         kernels.moe_plan(sorted_pair, tiles, n_tiles, chosen, pairs, self.experts)
         act = ws.get("moe_act", (pairs, self.inter), self.dtype)
         kernels.moe_expert_up(act, x, self.w_up, tiles, n_tiles, sorted_pair, pairs, top, self.activation,
-                              gated=self.gated)
+                              gated=self.gated, limit=self.limit, input_weight=weight if self.weigh_input else None)
         pair_out = ws.get("moe_pair_out", (pairs, self.hidden), torch.float32)
-        kernels.moe_expert_down(pair_out, act, self.w_down, tiles, n_tiles, sorted_pair, weight, pairs)
-        out = ws.get("mlp_down", (t, self.hidden), self.dtype)
-        kernels.moe_combine(out, pair_out, t, top)
+        kernels.moe_expert_down(pair_out, act, self.w_down, tiles, n_tiles, sorted_pair,
+                                None if self.weigh_input else weight, pairs)
+        add = None
+        if self.shared is not None:
+            self.shared.product_image = self.product_image
+            add = self.shared.forward(x, ctx)
+        out = ws.get("moe_out", (t, self.hidden), self.dtype)
+        kernels.moe_combine(out, pair_out, t, top, add=add)
         return out

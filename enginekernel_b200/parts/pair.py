@@ -9,14 +9,21 @@ forms it on its way through the row (the ``sandwich`` block takes pairs).
 Each side works in scratch buffers of its own, so that the first result outlives the second mixer's run.
 
 Parameters: ``first``, ``second`` (PartSpecs of role mixer), ``weight_first``, ``weight_second``.
+
+With ``result_eps`` (and the tensors ``first_gain``, ``second_gain`` [``hidden_size``]) both results are RMS-normed over
+their width before the sum, and the part hands on a :class:`~enginekernel_b200.parts.base.NormedPair` instead; the
+two weights are then one (``weight_first`` = ``weight_second``).
 """
 
 from __future__ import annotations
 
 import dataclasses
 
+import torch
+
 from ..registry import lookup_part, register_part
-from .base import Mixer, WeightedPair
+from .base import Mixer, NormedPair, WeightedPair
+from .spec import TensorSpec
 
 
 class _SideWorkspace:
@@ -43,12 +50,18 @@ class MixerPair(Mixer):
         out = []
         for side in cls._sides(spec):
             out += lookup_part("mixer", side.kind).tensors(side)
+        if spec.params.get("result_eps") is not None:
+            out += [TensorSpec(spec.weights[n], (spec.params["hidden_size"],), "gain") for n in ("first_gain", "second_gain")]
         return out
 
     def __init__(self, spec, dtype, device):
         super().__init__(spec, dtype, device)
         self.sides = [lookup_part("mixer", s.kind)(s, dtype, device) for s in self._sides(spec)]
         self.weights = (float(self.param("weight_first")), float(self.param("weight_second")))
+        self.result_eps = spec.params.get("result_eps")
+        self.first_gain = self.second_gain = None
+        if self.result_eps is not None and self.weights[0] != self.weights[1]:
+            raise ValueError("mixer_pair: results that are normed first are summed with one weight")
         if any(s.cache_spec() is None for s in self.sides):
             raise ValueError("mixer_pair: both mixers must keep something per sequence")
 
@@ -61,6 +74,9 @@ class MixerPair(Mixer):
     def load(self, tensors):
         for s in self.sides:
             s.load(tensors)
+        if self.result_eps is not None:
+            self.first_gain = tensors[self.spec.weights["first_gain"]].to(torch.float32).contiguous()
+            self.second_gain = tensors[self.spec.weights["second_gain"]].to(torch.float32).contiguous()
 
     def prepare(self, max_positions):
         for s in self.sides:
@@ -80,4 +96,6 @@ class MixerPair(Mixer):
         for i, (side, view) in enumerate(zip(self.sides, entry)):
             sub = dataclasses.replace(ctx, workspace=_SideWorkspace(ctx.workspace, f"side{i}_"))
             results.append(side.forward(x, sub, view, writes_cache))
+        if self.result_eps is not None:
+            return NormedPair(results[0], self.first_gain, results[1], self.second_gain, self.result_eps, self.weights[0])
         return WeightedPair(results[0], self.weights[0], results[1], self.weights[1])

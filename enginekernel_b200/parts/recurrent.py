@@ -1,5 +1,6 @@
-"""Two recurrent mixers with a decay per head and token, over one scan kernel, and one with a decay per
-channel and no matrix state (``gated_linear_recurrence``, described at its class).
+"""Two recurrent mixers with a decay per head and token, over one scan kernel, one over the same kernel whose
+decays are constants of the heads (``fixed_decay_memory``), and one with a decay per channel and no matrix state
+(``gated_linear_recurrence``; both described at their classes).
 
 Both keep a matrix S [key size, value size] per head and sequence in 32-bit and update it token by token,
 
@@ -182,6 +183,64 @@ class MatrixMemory(Mixer):
                            n_tokens=t)
         y = ws.get("attn_out", (t, nh * e), self.dtype)
         kernels.xlstm_out(y, o, m_run, proj, col_g, self.norm_w, self.eps, d ** -0.5, ctx.positions, t, nh, e)
+        return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
+
+
+@register_part("mixer", "fixed_decay_memory")
+class FixedDecayMemory(Mixer):
+    """Linear attention whose heads forget at fixed rates (Lightning attention).  H heads, key size d, value size e:
+
+        q = silu(W_q h), k = silu(W_k h), v = silu(W_v h)
+        S_t = decay_head S_(t-1) + k_t v_t^T;   o_t = S_t^T q_t          (no other scale; S from zero, 32-bit)
+        y = o / rms(o) * w * sigmoid(W_g h), the mean over all heads together;   out = W_o y
+
+    Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``v_dim``, ``decay`` (H numbers), ``eps``.  Tensors:
+    ``q``, ``k`` [H d, hidden], ``v``, ``g`` [H e, hidden], ``norm`` [H e], ``o`` [hidden, H e]."""
+
+    @classmethod
+    def tensors(cls, spec):
+        p, w = spec.params, spec.weights
+        hid, nh, d, e = p["hidden_size"], p["num_heads"], p["head_dim"], p["v_dim"]
+        return [TensorSpec(w["q"], (nh * d, hid)), TensorSpec(w["k"], (nh * d, hid)), TensorSpec(w["v"], (nh * e, hid)),
+                TensorSpec(w["g"], (nh * e, hid)), TensorSpec(w["norm"], (nh * e,), "gain"),
+                TensorSpec(w["o"], (hid, nh * e))]
+
+    def __init__(self, spec, dtype, device):
+        super().__init__(spec, dtype, device)
+        g = lambda n: int(self.param(n))
+        self.hidden, self.num_heads, self.head_dim, self.v_dim = g("hidden_size"), g("num_heads"), g("head_dim"), g("v_dim")
+        self.eps = float(self.param("eps"))
+        self.decay = [float(x) for x in self.param("decay")]
+        if len(self.decay) != self.num_heads:
+            raise ValueError("fixed_decay_memory: one decay per head")
+        self.rows = kernels.decay_scan_rows(self.head_dim)
+        self.s_values = self.num_heads * self.v_dim * self.rows
+        self.w_in = self.w_o = self.norm_w = self.a = self.b = None
+
+    def cache_spec(self):
+        return CacheSpec("state", shape=(-(-self.s_values // 4) * 4,))
+
+    def load(self, tensors):
+        w, f32 = self.spec.weights, torch.float32
+        rows = [tensors[w[n]] for n in ("q", "k", "v", "g")]
+        self.w_in = _padded_rows(rows, self.hidden).to(self.dtype).contiguous()
+        self.norm_w = tensors[w["norm"]].to(f32).contiguous()
+        self.w_o = tensors[w["o"]].to(self.dtype).contiguous()
+        self.a = torch.tensor(self.decay, dtype=f32, device=self.device)
+        self.b = torch.ones_like(self.a)
+
+    def forward(self, x, ctx, entry, writes_cache=True):
+        t, ws, f32 = ctx.n_tokens, ctx.workspace, torch.float32
+        nh, d, e = self.num_heads, self.head_dim, self.v_dim
+        proj = linear(x, self.w_in, ctx, "fdm_in", n_rows=t, out_dtype=f32, wide_f32="library")
+        width = nh * (2 * d + e)                             # q | k | v, and the gate behind them
+        qkv = ws.get("fdm_qkv", (t, width), f32)
+        kernels.bias_act(qkv, proj, None, "silu", n_rows=t)
+        o = ws.get("scan_o", (t, nh * e), f32)
+        kernels.decay_scan(o, qkv, qkv[:, nh * d:], qkv[:, 2 * nh * d:], self.a, self.b, entry.state, ctx.cu_seqlens,
+                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache, n_tokens=t)
+        y = ws.get("attn_out", (t, nh * e), self.dtype)
+        kernels.norm_gate_out(y, o, proj, width, self.norm_w, self.eps, ctx.positions, t)
         return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
 
 

@@ -20,6 +20,16 @@ from .base import PositionEncoding
 _TABLES: Dict[tuple, tuple] = {}
 
 
+def neighbours_to_halves(dim: int, rotary_dim: int) -> torch.Tensor:
+    """Order of a head's values that turns the pairs (2i, 2i + 1) of its first ``rotary_dim`` values into
+    the pairs (i, i + rotary_dim / 2): new[i] = old[order[i]].  Scores do not change when the rows of the query and
+    key projections (and their biases and gains) are reordered alike, so a design that turns neighbours runs on the
+    kernels that turn halves."""
+    even = list(range(0, rotary_dim, 2))
+    odd = list(range(1, rotary_dim, 2))
+    return torch.tensor(even + odd + list(range(rotary_dim, dim)), dtype=torch.long)
+
+
 @register_part("position", "rope_neox")
 class RopeNeox(PositionEncoding):
     def __init__(self, spec, dtype, device):
@@ -109,5 +119,51 @@ class RopeStretched(PositionEncoding):
                 _TABLES.clear()
             _TABLES[key] = ((ang.cos() * mult).to(torch.float32).to(self.device).contiguous(),
                             (ang.sin() * mult).to(torch.float32).to(self.device).contiguous())
+        self.cos, self.sin = _TABLES[key]
+        self.num_positions = max_positions
+
+
+@register_part("position", "rope_by_wavelength")
+class RopeByWavelength(PositionEncoding):
+    """NeoX-paired rotation that slows a dimension down by its wavelength (the scaling of Llama 3.1).
+
+    With f_i = theta^(-2i/rot) and wavelength l = 2 pi / f: f stays where l < original / high, becomes f / factor
+    where l > original / low, and between the two (1 - s) f / factor + s f with s = (original / l - low) /
+    (high - low).  Parameters: ``rotary_dim`` (rot), ``theta``, and ``factor``, ``low``, ``high``, ``original``
+    (without ``factor``: the plain rotation).  Worked out in 64-bit on the host, kept in 32-bit."""
+
+    def __init__(self, spec, dtype, device):
+        super().__init__(spec, dtype, device)
+        self.rotary_dim = int(self.param("rotary_dim"))
+        self.theta = float(self.param("theta"))
+        if self.rotary_dim % 2 or self.rotary_dim < 0:
+            raise ValueError(f"rotary_dim {self.rotary_dim} must be even")
+        self.scaling = None
+        if spec.params.get("factor") is not None:
+            self.scaling = tuple(float(self.param(n)) for n in ("factor", "low", "high", "original"))
+            if not (all(v > 0 for v in self.scaling) and self.scaling[2] > self.scaling[1]):
+                raise ValueError("rope_by_wavelength: factor, low, high and original must be positive, high above low")
+        self.cos = self.sin = None
+        self.num_positions = 0
+
+    def frequencies(self):
+        """Angle per position of every pair, [rot/2] in 64-bit."""
+        import math
+        f = self.theta ** (-2.0 * torch.arange(self.rotary_dim // 2, dtype=torch.float64) / max(self.rotary_dim, 1))
+        if self.scaling is None:
+            return f
+        factor, low, high, original = self.scaling
+        turns = original * f / (2.0 * math.pi)               # original / wavelength
+        s = torch.clamp((turns - low) / (high - low), 0.0, 1.0)
+        return (1.0 - s) * f / factor + s * f
+
+    def prepare(self, max_positions: int) -> None:
+        key = ("by_wavelength", str(self.device), self.theta, self.rotary_dim, max_positions, self.scaling)
+        if key not in _TABLES:
+            ang = torch.outer(torch.arange(max_positions, dtype=torch.float64), self.frequencies())
+            if len(_TABLES) > 8:
+                _TABLES.clear()
+            _TABLES[key] = (ang.cos().to(torch.float32).to(self.device).contiguous(),
+                            ang.sin().to(torch.float32).to(self.device).contiguous())
         self.cos, self.sin = _TABLES[key]
         self.num_positions = max_positions

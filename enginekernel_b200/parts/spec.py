@@ -21,7 +21,8 @@ class TensorSpec:
     name: str
     shape: Tuple[int, ...]
     #: how the random-weights mode fills it: "linear" and "embedding" are N(0, std),
-    #: "gain" is 1 + N(0, std_gain); "int" tensors are integer tables
+    #: "gain" is 1 + N(0, std_gain), "around_zero" N(0, std_gain); "average" (weights of a sum over layers) is
+    #: N(0, std) with 1 added to the last value; "int" tensors are integer tables
     init: str = "linear"
     #: "float" tensors are computed with in the engine's dtype; "int" become int32
     numeric: str = "float"

@@ -417,7 +417,7 @@ def test_router_against_the_plain_one(experts, top):
         logits = rnd(70, experts, seed=experts + top, scale=scale)
         chosen = torch.empty(70, top, dtype=torch.int32, device=DEV)
         weight = torch.empty(70, top, device=DEV)
-        k.moe_route(chosen, weight, logits, 70, 1, 1, top, 1.0, among_chosen=True)
+        k.moe_route(chosen, weight, logits, 70, 1, 1, top, 1.0, weights="softmax_of_chosen")
         vals, idx = torch.topk(logits.double().cpu(), top, dim=-1)
         assert torch.equal(chosen.cpu().long(), idx)
         assert rel(weight, torch.softmax(vals, -1)) <= 1e-5
