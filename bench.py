@@ -6,6 +6,7 @@
     python bench.py --design susalorn [--sizes 1b,2b-dense] [--layers L] [--batch B] [--skip-kernels]
     python bench.py --design bolelix [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
     python bench.py --design musavik [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
+    python bench.py --design kamosun [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
 
 The shapes and workloads are the ones BASELINE.json names (its configs[2], [3], [4]):
 
@@ -35,6 +36,9 @@ count and experts.
 ``--design musavik`` measures the Musavik decoder (two gated linear recurrences, then attention with mixed heads
 beside a delta rule, every layer with norms on both sides of its sublayers and a dense feed-forward) next to the
 Bolelix decoder of the same width and layer count.
+``--design kamosun`` measures the Kamosun decoder (a pair of full attention and fixed-decay memory, then three layers of
+chunked attention, one of which reads another's keys, all with gated results, averages over the depth and routed
+experts beside a shared one) next to the Bolelix decoder of the same width, layer count and experts.
 One line of JSON is printed.  The inputs of a step (gigabytes of weights) are larger than
 the L2.
 
@@ -48,6 +52,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import re
 import shutil
@@ -475,9 +480,54 @@ def musavik_configs(size: dict, layers: int, context: int):
     return musavik, bolelix_configs(BOLELIX_SIZES[size["beside"]], layers, context)[0]
 
 
+# Kamosun at sizes that resemble real layers, beside the Bolelix decoder - the closest design here: it too runs both
+# sublayers of a layer side by side on the same stream, mixes attention (with keys shared between layers) with
+# recurrences over the decay scan, and has gated experts - at the same width, layer count, head sizes and experts.
+# Layers in turn: the pair of full attention and fixed-decay memory, chunked attention, chunked attention that reads
+# the keys of the layer before it, chunked attention; the first layer's feed-forward is dense.
+KAMOSUN_SIZES = {
+    "1b": dict(width=2048, vocab=128256,
+               left=dict(heads=16, kv_heads=8, dim=128, vdim=128, rot=128), right=dict(heads=16, dim=128, vdim=128),
+               attention=dict(heads=16, kv_heads=8, dim=128, vdim=128, rot=128, chunk=1024),
+               moe=dict(experts=32, ff=1024, top=4, shared=1024), dense=6144, beside="1b"),
+    "2b": dict(width=2560, vocab=151936,
+               left=dict(heads=10, kv_heads=10, dim=128, vdim=256, rot=128), right=dict(heads=20, dim=128, vdim=128),
+               attention=dict(heads=20, kv_heads=10, dim=128, vdim=128, rot=64, chunk=512),
+               moe=dict(experts=16, ff=1536, top=2, shared=2048), dense=7680, beside="2b"),
+}
+
+
+def kamosun_configs(size: dict, layers: int, context: int):
+    """(Kamosun configuration, Bolelix configuration) of one size."""
+    from enginekernel_b200.config.kamosun import KamosunConfig
+
+    def attention(at, **more):
+        return dict({"dim": at["dim"], "vdim": at["vdim"], "heads": at["heads"], "kv_heads": at["kv_heads"],
+                     "scale": at["dim"] ** -0.5, "rot": {"base": 1000000.0, "dims": at["rot"]}}, **more)
+
+    at, right, m = size["attention"], size["right"], size["moe"]
+    left = attention(size["left"], softcap=30.0)
+    left["rot"]["scaling"] = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}
+    decay = [math.exp(-2.0 ** (-8.0 * (h + 1) / right["heads"])) for h in range(right["heads"])]
+    moe = {"kind": "moe", "expert": {"ff": m["ff"], "limit": 7.0}, "shared": {"ff": m["shared"], "limit": 7.0},
+           "router": {"experts": m["experts"], "top": m["top"]}}
+    made = []
+    for i in range(layers):
+        if i % 4 == 0:
+            mixer = {"left": left, "right": dict(right, decay=decay)}
+        else:
+            mixer = attention(at, mask={"size": at["chunk"]}, **({"kv_from": i - 1} if i % 4 == 2 else {}))
+        made.append({"type": "attention" if i % 4 else "parallel", "mixer": mixer,
+                     "mlp": moe if i else {"kind": "dense", "ff": size["dense"], "limit": 7.0}})
+    kamosun = KamosunConfig.from_dict({"architecture": "Kamosun", "vocab": size["vocab"], "width": size["width"],
+                                       "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": made})
+    return kamosun, bolelix_configs(BOLELIX_SIZES[size["beside"]], layers, context)[0]
+
+
 #: design -> (sizes, configurations of one size, the design it is measured beside)
 DESIGNS = {"lopazen": (DESIGN_SIZES, design_configs, "qwen3"), "susalorn": (SUSALORN_SIZES, susalorn_configs, "qwen3"),
-           "bolelix": (BOLELIX_SIZES, bolelix_configs, "susalorn"), "musavik": (MUSAVIK_SIZES, musavik_configs, "bolelix")}
+           "bolelix": (BOLELIX_SIZES, bolelix_configs, "susalorn"), "musavik": (MUSAVIK_SIZES, musavik_configs, "bolelix"),
+           "kamosun": (KAMOSUN_SIZES, kamosun_configs, "bolelix")}
 
 
 def measure_design(cfg, vocab, batch, prompt_len, context, steps, warmup, pk, with_kernels):
@@ -603,9 +653,9 @@ def main(argv=None) -> int:
     ap.add_argument("--skip-kernels", action="store_true", help="leave out the per-kernel tables")
     ap.add_argument("--prefill-seqs", type=int, default=1,
                     help="sequences of 2,048 tokens in the prompt step of the per-kernel table")
-    ap.add_argument("--design", default="", choices=["", "lopazen", "susalorn", "bolelix", "musavik"],
+    ap.add_argument("--design", default="", choices=["", "lopazen", "susalorn", "bolelix", "musavik", "kamosun"],
                     help="instead of the default workload: this design beside the Qwen3 decoder (bolelix: beside "
-                         "the Susalorn decoder; musavik: beside the Bolelix decoder) at equal layer sizes (prompt "
+                         "the Susalorn decoder; musavik, kamosun: beside the Bolelix decoder) at equal layer sizes (prompt "
                          "step, decode step, per-kernel tables)")
     ap.add_argument("--sizes", default="", help="with --design: comma-separated names of DESIGN_SIZES")
     args = ap.parse_args(argv)

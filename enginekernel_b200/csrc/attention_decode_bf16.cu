@@ -17,7 +17,7 @@
 // the window; their 16-key units are walked before the window's, by the first split.  `gate`, if given,
 // holds one value per token and query head (row stride `gate_stride`): the head's output is multiplied
 // by its sigmoid where the output is written.
-// `chunk` > 0 (instead of a window): a token sees the keys of its own chunk only.  `cap_out` > 0: scores pass
+// `chunk` > 0 (instead of a window): a token sees the keys of its own chunk only.  CAP: scores pass
 // a soft cap, cap * tanh(score / cap), before the softmax.
 // The reference's counterpart is the Triton split-K flash-decoding kernel with the group
 // padded to 16 rows and tiles staged through shared memory (engine/ek_kernels.py:534-615,
@@ -67,7 +67,7 @@ attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_st
                              float* __restrict__ part_acc, float* __restrict__ part_ml,
                              float sink_log2, const float* __restrict__ sinks, int keep_first,
                              const bf16* __restrict__ gate, int gate_stride, int cross,
-                             float* __restrict__ out32, int chunk, float cap_in, float cap_out) {
+                             float* __restrict__ out32, int chunk, SoftCap cap) {
   constexpr int D = DCH * 32;
   extern __shared__ float smem[];              // [warps][16][D] accumulators, then [warps][16][2]
   float* o_s = smem;
@@ -174,7 +174,7 @@ attention_decode_bf16_kernel(bf16* __restrict__ out, const bf16* q, int q_row_st
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + 8 * j + 2 * tq + (e & 1);
-          const float sc = CAP ? cap_out * tanh_by_exp(s[j][e] * cap_in) : s[j][e] * scale_log2;
+          const float sc = CAP ? capped_log2(s[j][e], cap) : s[j][e] * scale_log2;
           const float v = (key >= m_lo && key <= m_hi) ? sc : -INFINITY;
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -335,7 +335,7 @@ static int launch_dch(bf16* out, const bf16* q, int q_row_stride, const int* pos
                              row_blocks, scale * 1.4426950408889634f, window, n_splits,
                              keys_per_split, part_acc, part_ml, sink * 1.4426950408889634f, sinks,
                              window > 0 ? keep_first : 0, gate, gate_stride, cross, out32, chunk,
-                             CAP ? scale / softcap : 0.f, CAP ? softcap * 1.4426950408889634f : 0.f);
+                             soft_cap(scale, softcap));
   if (e != cudaSuccess || n_splits == 1) return (int)e;
   dim3 cgrid(n_tokens, n_q_heads * cross);
   return (int)launch_pdl(attention_decode_combine_kernel, cgrid, dim3(64), 0, stream, out,

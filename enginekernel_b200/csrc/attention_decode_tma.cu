@@ -69,8 +69,7 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
                             const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
-                            int window, int* status, float sink_log2, int chunk, float cap_in,
-                            float cap_out) {
+                            int window, int* status, float sink_log2, int chunk, SoftCap cap) {
   constexpr int DB = D / 64;                       // 64-wide (128-byte) blocks of the head dimension
   constexpr uint32_t kSub = EK_PAGE * 128;         // one [64 keys x 64 dims] sub-tile: 8 KB
   constexpr uint32_t kStage = 2 * DB * kSub;       // K tile + V tile
@@ -205,7 +204,7 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int key = key0 + 8 * j + 2 * tq + (e & 1);
-              const float score = cap_out > 0.f ? cap_out * tanh_by_exp(sc[j][e] * cap_in) : sc[j][e] * scale_log2;
+              const float score = cap.c > 0.f ? capped_log2(sc[j][e], cap) : sc[j][e] * scale_log2;
               const float v = (key >= lo && key <= hi) ? score : -INFINITY;
               sc[j][e] = v;
               mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -403,12 +402,11 @@ static int launch_dt(bf16* out, const bf16* q, int q_row_stride, const int* posi
                                      q_row_stride, positions, token_slot, mk, mv, block_table,
                                      table_stride, n_kv_heads, n_q_heads,
                                      scale * 1.4426950408889634f, window, status,
-                                     sink * 1.4426950408889634f, chunk, softcap > 0.f ? scale / softcap : 0.f,
-                                     softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
+                                     sink * 1.4426950408889634f, chunk, soft_cap(scale, softcap));
   return (int)launch_pdl(kernel, grid, dim3(kDtThreads), smem, stream, out, q, q_row_stride, positions,
                          token_slot, mk, mv, block_table, table_stride, n_kv_heads, n_q_heads,
                          scale * 1.4426950408889634f, window, status, sink * 1.4426950408889634f, chunk,
-                         softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
+                         soft_cap(scale, softcap));
 }
 
 }  // namespace ek

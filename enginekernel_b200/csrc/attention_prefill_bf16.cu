@@ -15,7 +15,7 @@
 // given, holds one value per token and query head (row stride `gate_stride`): the head's output is
 // multiplied by its sigmoid.
 // `chunk` > 0 (instead of a window): a row sees the keys of its own chunk only, chunks being counted from the
-// sequence's first position.  `cap_out` > 0: scores pass a soft cap, cap * tanh(score / cap), before the softmax.
+// sequence's first position.  `cap`: scores pass a soft cap, cap * tanh(score / cap), before the softmax.
 // Tiles are found from cu_seqlens on the device (no host-built schedule).
 // The reference's counterpart is a Triton kernel over a padded rectangle, 128x128 tiles,
 // probabilities rounded to bfloat16 before P.V as here (engine/ek_kernels.py:166-221),
@@ -67,7 +67,7 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
                               int n_q_heads, float scale_log2, int window, int tok_per_tile,
                               float sink_log2, const float* __restrict__ sinks, int keep_first,
                               const bf16* __restrict__ gate, int gate_stride, int cross,
-                              float* __restrict__ out32, int chunk, float cap_in, float cap_out) {
+                              float* __restrict__ out32, int chunk, SoftCap cap) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int tile_info[3];                 // first token (packed index), tokens, sequence
   const int D = cache.head_dim;
@@ -210,7 +210,7 @@ attention_prefill_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ q
       for (int j = 0; j < kPfKeys / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          float v = cap_out > 0.f ? cap_out * tanh_by_exp(s[j][e] * cap_in) : s[j][e] * scale_log2;
+          float v = cap.c > 0.f ? capped_log2(s[j][e], cap) : s[j][e] * scale_log2;
           if (need_mask) {
             const int key = key0 + 8 * j + 2 * tq + (e & 1);
             const int p = e < 2 ? pos_lo : pos_hi;
@@ -346,7 +346,7 @@ static int launch_dmax(bf16* out, const bf16* q, int q_row_stride, const int* po
       out, q, q_row_stride, positions, token_slot, cu_seqlens, n_seqs, cache, n_q_heads,
       scale * 1.4426950408889634f, window, tok_per_tile, sink * 1.4426950408889634f, sinks,
       window > 0 ? keep_first : 0, gate, gate_stride, cross, out32, chunk,
-      softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
+      soft_cap(scale, softcap));
   EK_RETURN_LAUNCH_STATUS();
 }
 

@@ -67,9 +67,13 @@ __device__ __forceinline__ float2 add2(float2 a, float2 b) {
   return d;
 }
 
-// CAP: scores pass a soft cap before the softmax, cap tanh(score / cap): `cap_in` is scale / cap and
-// `scale_log2` then stands for cap log2(e), which multiplies the tanh.  `chunk` > 0 (instead of a window): a
+// CAP: scores pass a soft cap before the softmax, cap tanh(score / cap).  Capped scores lie within [-cap, cap], so
+// up to a cap of 40 (kBoundedCap) the exponentials need no running maximum: e^40 times any number of keys fits
+// 32 bits and e^-40 is far from the smallest bfloat16; beyond it the maximum is kept as without a cap.
+// `chunk` > 0 (instead of a window): a
 // row sees the keys of its own chunk of positions only.
+constexpr float kBoundedCap = 40.f * 1.4426950408889634f;
+
 template <int D, bool CAP>
 __global__ void __launch_bounds__(kFaThreads, 2)
 attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUtensorMap map_q,
@@ -78,7 +82,7 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
                             int window, int tok_per_tile, int* status, float sink_log2, int chunk,
-                            float cap_in) {
+                            SoftCap cap) {
   constexpr int DB = D / 64;                       // 64-wide blocks of the head dimension
   constexpr uint32_t kSub = kFaKeys * 128;         // one [64 x 64] bfloat16 sub-tile: 8 KB
   constexpr uint32_t kTmemCols = 256;
@@ -222,7 +226,8 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
 
   // ------------------------------------------------------------------------ softmax rows
   constexpr float kLazy = 8.f;                     // raise the reference maximum above 2^8 only
-  float m_ref = -INFINITY, l_run = 0.f;            // the reference is in units of log2(e)/scale
+  const bool bounded = CAP && cap.c <= kBoundedCap;
+  float m_ref = bounded ? 0.f : -INFINITY, l_run = 0.f;   // the reference is in units of log2(e)/scale
   const int r = tid;                               // row = TMEM lane (softmax threads)
   const uint32_t lane_addr = tmem_base + ((uint32_t)((warp & 3) * 32) << 16);
   if (tid < kFaRows) {
@@ -254,15 +259,17 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
       };
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // of the raw scores
       float sc[32];                                // (the scale is positive)
-      load_half(1, sc);
+      if (!CAP || !bounded) {
+        load_half(1, sc);
 #pragma unroll
-      for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sc[i]);
-      load_half(0, sc);
+        for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sc[i]);
+        load_half(0, sc);
 #pragma unroll
-      for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sc[i]);
+        for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sc[i]);
+      }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      if (CAP && mx > -INFINITY) mx = tanh_by_exp(mx * cap_in);   // (monotonic: the maximum's cap is the caps' maximum)
-      mx *= scale_log2;
+      if (CAP) mx = mx > -INFINITY ? capped_log2(mx, cap) : mx;   // (monotonic: the maximum's cap is the caps' maximum)
+      else mx *= scale_log2;
       // tcgen05.ld/st are warp-wide: if any row of the warp raises its reference, the whole warp
       // rescales (rows that keep theirs multiply by 1)
       const bool raise = mx > m_ref + kLazy;       // also the first page with a visible key
@@ -288,22 +295,34 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
         m_ref = mx;
       }
       const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
-      const float2 scale2 = make_float2(scale_log2, scale_log2), shift2 = make_float2(neg_m, neg_m);
+      // CAP: a capped score is c - 2c r with r = 1 / (2^(s k) + 1)
+      const float mul = CAP ? -2.f * cap.c : scale_log2, add = CAP ? cap.c + neg_m : neg_m;
+      const float2 scale2 = make_float2(mul, mul), shift2 = make_float2(add, add);
       float2 psum[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
       // P over the scores it came from: 32 keys are 16 columns; the first store is under way
       // while the second half is read again and computed
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
-        if (h == 1) load_half(1, sc);              // columns 32..63: untouched by the P of keys 0..31
+        if (CAP) {                                 // (the raw scores, unmasked: what is not seen gets P = 0 below)
+          tmem_ld32_nowait(lane_addr + kColS + 64 * s + 32 * h, sc);
+          tmem_ld_wait();
+        } else if (h == 1) {
+          load_half(1, sc);                        // columns 32..63: untouched by the P of keys 0..31
+        }
         uint32_t w[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          if (CAP) {                               // (a masked score stays what it is)
-            sc[i] = sc[i] > -INFINITY ? tanh_by_exp(sc[i] * cap_in) : sc[i];
-            sc[i + 1] = sc[i + 1] > -INFINITY ? tanh_by_exp(sc[i + 1] * cap_in) : sc[i + 1];
+          if (CAP) {
+            sc[i] = soft_cap_sigmoid(sc[i], cap.k);
+            sc[i + 1] = soft_cap_sigmoid(sc[i + 1], cap.k);
           }
           const float2 a = fma2(make_float2(sc[i], sc[i + 1]), scale2, shift2);
-          const float2 p = make_float2(ex2_approx(a.x), ex2_approx(a.y));
+          float2 p = make_float2(ex2_approx(a.x), ex2_approx(a.y));
+          if (CAP && !full) {
+            const int key = key0 + 32 * h + i;
+            p.x = key <= pos_r && key >= first_r ? p.x : 0.f;
+            p.y = key + 1 <= pos_r && key + 1 >= first_r ? p.y : 0.f;
+          }
           psum[(i >> 1) & 1] = add2(psum[(i >> 1) & 1], p);
           __nv_bfloat162 hh = __floats2bfloat162_rn(p.x, p.y);
           w[i / 2] = *reinterpret_cast<uint32_t*>(&hh);
@@ -482,9 +501,9 @@ static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* til
   if (n_tiles > 65535) return EK_ERR_ARG;
   dim3 grid(n_kv_heads, n_tiles);
   return (int)launch_pdl(kernel, grid, dim3(kFaThreads), smem, stream, out, mq, tiles, mk, mv, block_table,
-                         table_stride, n_kv_heads, n_q_heads, (CAP ? softcap : scale) * 1.4426950408889634f,
+                         table_stride, n_kv_heads, n_q_heads, scale * 1.4426950408889634f,
                          window, tok_per_tile, status, sink * 1.4426950408889634f, chunk,
-                         CAP ? scale / softcap : 0.f);
+                         soft_cap(scale, softcap));
 }
 
 }  // namespace ek

@@ -13,7 +13,7 @@
 #include <unordered_set>
 
 #define EK_PAGE 64          // tokens per cache page (must match cache/pages.py)
-#define EK_MAX_HEAD_DIM 256
+#define EK_MAX_HEAD_DIM 512  // of the kernels that prepare heads and store them (attention kernels have limits of their own)
 
 #define EK_ERR_ARG (-2)      // a size the kernel does not take
 #define EK_EXPORT extern "C" __attribute__((visibility("default")))
@@ -120,9 +120,28 @@ __device__ __forceinline__ int first_key(int pos, int window, int chunk) {
   return window > 0 ? max(0, pos - window + 1) : 0;
 }
 
-// tanh for the soft cap of attention scores in the 16-bit kernels: 1 - 2 / (e^(2x) + 1), whose absolute error
-// is a few 32-bit roundings of 1 (the exponential overflows to infinity and the quotient to 0 for large x).
+// tanh as 1 - 2 / (e^(2x) + 1), whose absolute error is a few 32-bit roundings of 1: for 16-bit results.
 __device__ __forceinline__ float tanh_by_exp(float x) { return 1.f - __fdividef(2.f, __expf(fminf(2.f * x, 80.f)) + 1.f); }
+
+// The soft cap of attention scores in the 16-bit kernels, in units of log2: c tanh(x) with c = cap log2(e) and
+// x = score / cap, as c - 2c / (2^(s k) + 1) where k = 2 log2(e) scale / cap turns the raw product s into 2x log2(e).
+// (A large s makes the power infinite and the reciprocal 0.)
+struct SoftCap {
+  float k, c;                // c <= 0: no cap
+};
+inline SoftCap soft_cap(float scale, float cap) {
+  if (!(cap > 0.f)) return SoftCap{0.f, 0.f};
+  return SoftCap{2.f * 1.4426950408889634f * scale / cap, cap * 1.4426950408889634f};
+}
+__device__ __forceinline__ float soft_cap_sigmoid(float s, float k) {      // 1 / (2^(s k) + 1)
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * k));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return r;
+}
+__device__ __forceinline__ float capped_log2(float s, SoftCap cap) {
+  return fmaf(-2.f * cap.c, soft_cap_sigmoid(s, cap.k), cap.c);
+}
 
 // Programmatic dependent launch: a kernel launched with `launch_pdl` may start while the
 // kernel before it on the stream is still draining.  It must call `pdl_wait()` before it

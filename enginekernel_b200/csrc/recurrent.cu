@@ -839,7 +839,8 @@ namespace ek {
 template <typename T>
 __global__ void __launch_bounds__(1024)
 norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float* __restrict__ proj, int proj_stride,
-                     int col_g, const float* __restrict__ w, float eps, const int* __restrict__ positions, int inner) {
+                     int col_g, const float* __restrict__ w, float eps, const int* __restrict__ positions, int inner,
+                     int vec) {
   __shared__ float scratch[33];
   pdl_launch_dependents();
   pdl_wait();
@@ -847,6 +848,35 @@ norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float
   if (positions[t] < 0) return;
   const float* row = o + t * inner;
   const float* gate = proj + t * proj_stride + col_g;
+  constexpr int kKeep4 = kOutKeep / 4;
+  if (vec && inner <= (int)blockDim.x * kOutKeep) {    // four neighbours a thread, everything fetched before the sum
+    float4 u4[kKeep4], g4[kKeep4];
+    float s4 = 0.f;
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m) {
+      const int i = (threadIdx.x + m * blockDim.x) * 4;
+      u4[m] = g4[m] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < inner) {
+        u4[m] = *reinterpret_cast<const float4*>(row + i);
+        g4[m] = *reinterpret_cast<const float4*>(gate + i);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m)
+      s4 += u4[m].x * u4[m].x + u4[m].y * u4[m].y + u4[m].z * u4[m].z + u4[m].w * u4[m].w;
+    const float rstd4 = rsqrtf(block_sum(s4, scratch) / (float)inner + eps);
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m) {
+      const int i = (threadIdx.x + m * blockDim.x) * 4;
+      if (i >= inner) continue;
+      const float4 w4 = *reinterpret_cast<const float4*>(w + i);
+      Vec4<T>::store(y + t * inner + i, make_float4(u4[m].x * rstd4 * w4.x * sigmoid_f(g4[m].x),
+                                                    u4[m].y * rstd4 * w4.y * sigmoid_f(g4[m].y),
+                                                    u4[m].z * rstd4 * w4.z * sigmoid_f(g4[m].z),
+                                                    u4[m].w * rstd4 * w4.w * sigmoid_f(g4[m].w)));
+    }
+    return;
+  }
   float u[kOutKeep], ss = 0.f;
 #pragma unroll
   for (int m = 0; m < kOutKeep; ++m) {           // the first values of a thread wait in registers
@@ -885,9 +915,11 @@ norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float
                                           int inner, cudaStream_t stream) {                                    \
     if (n_tokens <= 0) return 0;                                                                               \
     if (inner <= 0) return EK_ERR_ARG;                                                                         \
-    const int threads = inner >= 4096 ? 1024 : inner <= 256 ? 64 : (inner / 4 + 31) / 32 * 32;                 \
+    const int threads = inner >= 8192 ? 1024 : inner <= 512 ? 64 : (inner / 8 + 31) / 32 * 32;                 \
+    const int vec = inner % 4 == 0 && proj_stride % 4 == 0 && col_g % 4 == 0 && ((uintptr_t)y & 7) == 0 &&     \
+                    (((uintptr_t)o | (uintptr_t)proj | (uintptr_t)w) & 15) == 0;                               \
     return (int)ek::launch_pdl(ek::norm_gate_out_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (T*)y, o, \
-                               proj, proj_stride, col_g, w, eps, positions, inner);                            \
+                               proj, proj_stride, col_g, w, eps, positions, inner, vec);                       \
   }                                                                                                            \
   EK_EXPORT int ek_xlstm_out_##SUFFIX(void* y, const float* o, const float* m_run, const float* proj,          \
                                       int proj_stride, int col_g, const float* w, float eps, float q_scale,    \

@@ -232,17 +232,17 @@ __global__ void qk_rope_unit_kv_kernel(T* rows, int row_stride, int k_col, int v
 // and a head costs a lane two multiply-adds and one multiply per value:
 //     y_lo = rstd * (x_lo * (g_lo cos) - x_hi * (g_hi sin)),   y_hi = rstd * (x_hi * (g_hi cos) + x_lo * (g_lo sin))
 // which is gain * x * rstd rotated, with the 32-bit products taken in another order.  All loads of
-// a token are issued before the first use.
+// a token are issued before the first use.  BIAS: biases of the projections (QkExtras) come first.
 constexpr int kWideThreads = 256;
 constexpr int kWidePasses = 4;
 
-template <int D>
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(kWideThreads, 4)
 qk_norm_rope_kv_wide_kernel(bf16* qkv, int row_stride, const float* __restrict__ q_gain,
                             const float* __restrict__ k_gain, const float* __restrict__ cos_tab,
                             const float* __restrict__ sin_tab, const int* positions,
                             const int* token_slot, PagedKV cache, int n_q_heads, float eps,
-                            int write_kv) {
+                            int write_kv, QkExtras ex) {
   constexpr int LPH = D / 8;                       // lanes a head
   constexpr int HPP = kWideThreads / LPH;          // heads a pass
   constexpr int half = D / 2;
@@ -320,7 +320,8 @@ qk_norm_rope_kv_wide_kernel(bf16* qkv, int row_stride, const float* __restrict__
         const int kv_head = is_k ? head - n_q_heads : head - n_q_heads - n_kv;
         dst = (bf16*)(is_k ? cache.k : cache.v) + page_base + (size_t)kv_head * EK_PAGE * D + d0;
       }
-      if (!is_q && !is_k) {
+      const float* bias = BIAS ? (is_q ? ex.q_bias : (is_k ? ex.k_bias : ex.v_bias)) : nullptr;
+      if (!is_q && !is_k && !bias) {
         *reinterpret_cast<uint2*>(dst) = raw_lo[p];
         *reinterpret_cast<uint2*>(dst + half) = raw_hi[p];
         continue;
@@ -335,6 +336,19 @@ qk_norm_rope_kv_wide_kernel(bf16* qkv, int row_stride, const float* __restrict__
           lo[2 * i] = f.x; lo[2 * i + 1] = f.y;
           hi[2 * i] = g.x; hi[2 * i + 1] = g.y;
         }
+      }
+      if (BIAS && bias) {
+        bias += (size_t)(is_q ? head : (is_k ? head - n_q_heads : head - n_q_heads - n_kv)) * D;
+        const float4 bl = *reinterpret_cast<const float4*>(bias + d0), bh = *reinterpret_cast<const float4*>(bias + half + d0);
+        lo[0] += bl.x; lo[1] += bl.y; lo[2] += bl.z; lo[3] += bl.w;
+        hi[0] += bh.x; hi[1] += bh.y; hi[2] += bh.z; hi[3] += bh.w;
+      }
+      if (BIAS && !is_q && !is_k) {                // a value head with its bias
+        __nv_bfloat162 v0 = __floats2bfloat162_rn(lo[0], lo[1]), v1 = __floats2bfloat162_rn(lo[2], lo[3]);
+        __nv_bfloat162 v2 = __floats2bfloat162_rn(hi[0], hi[1]), v3 = __floats2bfloat162_rn(hi[2], hi[3]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&v0), *reinterpret_cast<uint32_t*>(&v1));
+        *reinterpret_cast<uint2*>(dst + half) = make_uint2(*reinterpret_cast<uint32_t*>(&v2), *reinterpret_cast<uint32_t*>(&v3));
+        continue;
       }
       float rstd = 1.f;
       if (is_q ? q_norm : k_norm) {
@@ -486,14 +500,14 @@ static int launch_prepare_wide(bf16* qkv, int row_stride, const float* q_gain, c
                          row_stride, q_gain, k_gain, positions, token_slot, cache, n_q_heads, eps, write_kv, ex);
 }
 
-template <int D>
+template <int D, bool BIAS = false>
 static int launch_wide(bf16* qkv, int row_stride, const float* q_gain, const float* k_gain,
                        const float* cos_tab, const float* sin_tab, const int* positions,
                        const int* token_slot, PagedKV cache, int n_tokens, int n_q_heads, float eps,
-                       int write_kv, cudaStream_t stream) {
-  return (int)launch_pdl(qk_norm_rope_kv_wide_kernel<D>, dim3(n_tokens), dim3(kWideThreads), 0, stream,
+                       int write_kv, cudaStream_t stream, QkExtras ex = QkExtras{}) {
+  return (int)launch_pdl(qk_norm_rope_kv_wide_kernel<D, BIAS>, dim3(n_tokens), dim3(kWideThreads), 0, stream,
                          qkv, row_stride, q_gain, k_gain, cos_tab, sin_tab, positions, token_slot, cache,
-                         n_q_heads, eps, write_kv);
+                         n_q_heads, eps, write_kv, ex);
 }
 
 // The wide form needs 16-byte rows and tables; one token a block pays once there are enough
@@ -553,6 +567,20 @@ static int launch(void* qkv, int row_stride, const float* q_gain, const float* k
                               cache, n_tokens, n_q_heads, eps, write_kv, stream);
     return launch_wide<256>(rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, positions, token_slot,
                             cache, n_tokens, n_q_heads, eps, write_kv, stream);
+  }
+  const bool biased_only = !plain && !padded && ex.q_temp_coef == 0.f && !ex.v_from_k &&
+                           (((uintptr_t)ex.q_bias | (uintptr_t)ex.k_bias | (uintptr_t)ex.v_bias) & 15) == 0;
+  if (biased_only && wide_takes<T>(qkv, row_stride, q_gain, k_gain, cos_tab, sin_tab, rot_dim, k_pages, v_pages,
+                                   n_tokens, head_dim)) {
+    bf16* rows = (bf16*)qkv;
+    if (head_dim == 64)
+      return launch_wide<64, true>(rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, positions, token_slot,
+                                   cache, n_tokens, n_q_heads, eps, write_kv, stream, ex);
+    if (head_dim == 128)
+      return launch_wide<128, true>(rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, positions, token_slot,
+                                    cache, n_tokens, n_q_heads, eps, write_kv, stream, ex);
+    return launch_wide<256, true>(rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, positions, token_slot,
+                                  cache, n_tokens, n_q_heads, eps, write_kv, stream, ex);
   }
   const int heads = n_q_heads + (ex.v_from_k ? 1 : 2) * n_kv_heads;
   dim3 grid(n_tokens, (heads + kRopeWarps - 1) / kRopeWarps);

@@ -18,7 +18,8 @@ from . import lib
 from .lib import Function, KernelError, count_extra_launches
 
 PAGE = 64                 # tokens per cache page; must equal EK_PAGE in csrc/common.cuh
-MAX_HEAD_DIM = 256
+MAX_HEAD_DIM = 256        # of the 16-bit attention kernels
+PREPARE_MAX_HEAD_DIM = 512      # of the kernels that norm, rotate and store heads; equals EK_MAX_HEAD_DIM in csrc/common.cuh
 GENERIC_MAX_HEAD_DIM = 1024     # the general attention kernel alone takes head sizes up to here
 
 _SUFFIX = {torch.float32: "f32", torch.bfloat16: "bf16"}
@@ -409,9 +410,9 @@ _rope_kv = _per_dtype("rope_kv", "ek_qk_norm_rope_kv",
 
 
 def check_head_dim(head_dim):
-    if not 1 <= head_dim <= MAX_HEAD_DIM:
-        raise KernelError(f"head size {head_dim} is not supported: the attention kernels take "
-                          f"head sizes up to {MAX_HEAD_DIM}")
+    if not 1 <= head_dim <= PREPARE_MAX_HEAD_DIM:
+        raise KernelError(f"head size {head_dim} is not supported: the kernels that prepare heads take "
+                          f"sizes up to {PREPARE_MAX_HEAD_DIM}")
 
 
 _qk_prepare = _per_dtype("rope_kv", "ek_qk_prepare_kv",
