@@ -69,7 +69,8 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
                             const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
-                            int window, int* status, float sink_log2, int chunk, SoftCap cap) {
+                            int window, int* status, float sink_log2, const float* __restrict__ sinks, int chunk,
+                            SoftCap cap) {
   constexpr int DB = D / 64;                       // 64-wide (128-byte) blocks of the head dimension
   constexpr uint32_t kSub = EK_PAGE * 128;         // one [64 keys x 64 dims] sub-tile: 8 KB
   constexpr uint32_t kStage = 2 * DB * kSub;       // K tile + V tile
@@ -304,7 +305,8 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
       }
       if (n_splits == 1) {
         // a sink: one more term exp(sink) in the denominator, with no value (-inf: none)
-        if (sink_log2 > -INFINITY && l > 0.f) l += exp2f(sink_log2 - m);
+        const float sk = sinks ? sinks[head0 + r] * 1.4426950408889634f : sink_log2;   // per head, if given
+        if (sk > -INFINITY && l > 0.f) l += exp2f(sk - m);
         out[((size_t)t * n_q_heads + head0 + r) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
       } else {
         const int owner = idx / run;
@@ -339,7 +341,8 @@ attention_decode_tma_kernel(bf16* __restrict__ out, const bf16* q, int q_row_str
           o += recv_o[sp * run + slot] * f;
         }
       }
-      if (sink_log2 > -INFINITY && l > 0.f) l += exp2f(sink_log2 - m);   // the sink, counted once
+      const float sk = sinks ? sinks[head0 + r] * 1.4426950408889634f : sink_log2;
+      if (sk > -INFINITY && l > 0.f) l += exp2f(sk - m);      // the sink, counted once
       out[((size_t)t * n_q_heads + head0) * D + idx] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
   }
@@ -352,7 +355,7 @@ static int launch_dt(bf16* out, const bf16* q, int q_row_stride, const int* posi
                      const int* token_slot, const void* k_pages, const void* v_pages,
                      long long page_rows, const int* block_table, int table_stride, int n_tokens,
                      int n_q_heads, int n_kv_heads, float scale, int window, int n_splits, int* status,
-                     float sink, int chunk, float softcap, cudaStream_t stream) {
+                     float sink, const float* sinks, int chunk, float softcap, cudaStream_t stream) {
   constexpr int STAGES = (D == 128 ? 3 : 6) * (DEEP ? 2 : 1);
   constexpr int DB = D / 64;
   constexpr size_t smem = 1024 + (size_t)STAGES * 2 * DB * EK_PAGE * 128 + 2 * STAGES * 8 +
@@ -402,10 +405,10 @@ static int launch_dt(bf16* out, const bf16* q, int q_row_stride, const int* posi
                                      q_row_stride, positions, token_slot, mk, mv, block_table,
                                      table_stride, n_kv_heads, n_q_heads,
                                      scale * 1.4426950408889634f, window, status,
-                                     sink * 1.4426950408889634f, chunk, soft_cap(scale, softcap));
+                                     sink * 1.4426950408889634f, sinks, chunk, soft_cap(scale, softcap));
   return (int)launch_pdl(kernel, grid, dim3(kDtThreads), smem, stream, out, q, q_row_stride, positions,
                          token_slot, mk, mv, block_table, table_stride, n_kv_heads, n_q_heads,
-                         scale * 1.4426950408889634f, window, status, sink * 1.4426950408889634f, chunk,
+                         scale * 1.4426950408889634f, window, status, sink * 1.4426950408889634f, sinks, chunk,
                          soft_cap(scale, softcap));
 }
 
@@ -418,10 +421,10 @@ EK_EXPORT int ek_attention_decode_tma_max_splits(int head_dim) {
   int clusters = 0;
   if (head_dim == 64)
     clusters = launch_dt<64, false, true>(nullptr, nullptr, 0, nullptr, nullptr, &clusters, &clusters, 64,
-                                          nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, 0, 0.f, nullptr);
+                                          nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, nullptr, 0, 0.f, nullptr);
   else if (head_dim == 128)
     clusters = launch_dt<128, false, true>(nullptr, nullptr, 0, nullptr, nullptr, &clusters, &clusters, 64,
-                                           nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, 0, 0.f, nullptr);
+                                           nullptr, 0, 1, 1, 1, 1.f, 0, 1, nullptr, -INFINITY, nullptr, 0, 0.f, nullptr);
   else
     return 0;
   return clusters >= 1 ? kDtMaxSplits : kDtPortableSplits;
@@ -431,15 +434,16 @@ EK_EXPORT int ek_attention_decode_tma_max_splits(int head_dim) {
 // the token's visible range); q rows 4-byte aligned; n_pages = pages in k_pages / v_pages
 // ([pages, kv heads, 64, head_dim]); `status` is one int on the device.  `sink`: score of a key
 // without a value that every query also sees (one more term in the softmax denominator);
-// -INFINITY for none.  `chunk` > 0 instead of a window: keys of the token's own chunk of positions only.
+// -INFINITY for none; `sinks` (may be null): one such score per query head, in place of `sink`.
+// `chunk` > 0 instead of a window: keys of the token's own chunk of positions only.
 // `softcap` > 0: scores become softcap tanh(score / softcap).
 EK_EXPORT int ek_attention_decode_tma(void* out, const void* q, int q_row_stride,
                                       const int* positions, const int* token_slot,
                                       const void* k_pages, const void* v_pages, int n_pages,
                                       const int* block_table, int table_stride, int n_tokens,
                                       int n_q_heads, int n_kv_heads, int head_dim, float scale,
-                                      int window, int n_splits, int* status, float sink, int chunk,
-                                      float softcap, cudaStream_t stream) {
+                                      int window, int n_splits, int* status, float sink,
+                                      const float* sinks, int chunk, float softcap, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
   if (chunk < 0 || (chunk > 0 && window > 0)) return EK_ERR_ARG;
@@ -453,8 +457,8 @@ EK_EXPORT int ek_attention_decode_tma(void* out, const void* q, int q_row_stride
 #define EK_DT(D_, DEEP_)                                                                          \
   return launch_dt<D_, DEEP_>((bf16*)out, (const bf16*)q, q_row_stride, positions, token_slot,     \
                               k_pages, v_pages, page_rows, block_table, table_stride, n_tokens,   \
-                              n_q_heads, n_kv_heads, scale, window, n_splits, status, sink, chunk,     \
-                              softcap, stream)
+                              n_q_heads, n_kv_heads, scale, window, n_splits, status, sink, sinks,     \
+                              chunk, softcap, stream)
   if (head_dim == 64) {
     if (deep) EK_DT(64, true);
     EK_DT(64, false);

@@ -81,8 +81,8 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
                             const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* block_table,
                             int table_stride, int n_kv_heads, int n_q_heads, float scale_log2,
-                            int window, int tok_per_tile, int* status, float sink_log2, int chunk,
-                            SoftCap cap) {
+                            int window, int tok_per_tile, int* status, float sink_log2,
+                            const float* __restrict__ sinks, int chunk, SoftCap cap) {
   constexpr int DB = D / 64;                       // 64-wide blocks of the head dimension
   constexpr uint32_t kSub = kFaKeys * 128;         // one [64 x 64] bfloat16 sub-tile: 8 KB
   constexpr uint32_t kTmemCols = 256;
@@ -346,7 +346,9 @@ attention_prefill_tc_kernel(bf16* __restrict__ out, const __grid_constant__ CUte
   if (!failed) {
     if (tid < kFaRows) {                           // whole warps: tcgen05.ld is warp-wide
       // a sink: one more term exp(sink) in the denominator, with no value (-inf: none)
-      if (sink_log2 > -INFINITY && l_run > 0.f) l_run += exp2f(sink_log2 - m_ref);
+      // (`sinks`: one score per query head instead of the same for all)
+      const float sk = sinks ? sinks[kv_head * group + r % group] * 1.4426950408889634f : sink_log2;
+      if (sk > -INFINITY && l_run > 0.f) l_run += exp2f(sk - m_ref);
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       const bool wide_out = ((uintptr_t)out & 31) == 0;     // rows of D values are then 32-byte aligned
       const int row = min(r, n_rows - 1);
@@ -475,8 +477,8 @@ template <int D, bool CAP>
 static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* tiles, int n_tiles, int n_tokens,
                      const void* k_pages, const void* v_pages, long long page_rows,
                      const int* block_table, int table_stride, int n_q_heads, int n_kv_heads,
-                     float scale, int window, int* status, float sink, int chunk, float softcap,
-                     cudaStream_t stream) {
+                     float scale, int window, int* status, float sink, const float* sinks, int chunk,
+                     float softcap, cudaStream_t stream) {
   const int group = n_q_heads / n_kv_heads;
   const int tok_per_tile = kFaRows / group;
   CUtensorMap mq, mk, mv;
@@ -502,7 +504,7 @@ static int launch_fa(bf16* out, const bf16* q, int q_row_stride, const int4* til
   dim3 grid(n_kv_heads, n_tiles);
   return (int)launch_pdl(kernel, grid, dim3(kFaThreads), smem, stream, out, mq, tiles, mk, mv, block_table,
                          table_stride, n_kv_heads, n_q_heads, scale * 1.4426950408889634f,
-                         window, tok_per_tile, status, sink * 1.4426950408889634f, chunk,
+                         window, tok_per_tile, status, sink * 1.4426950408889634f, sinks, chunk,
                          soft_cap(scale, softcap));
 }
 
@@ -534,8 +536,8 @@ EK_EXPORT int ek_attention_prefill_tc(void* out, const void* q, int q_row_stride
                                       const void* k_pages, const void* v_pages, int n_pages,
                                       const int* block_table, int table_stride, int n_q_heads,
                                       int n_kv_heads, int head_dim, float scale, int window,
-                                      int* status, float sink, int chunk, float softcap,
-                                      cudaStream_t stream) {
+                                      int* status, float sink, const float* sinks, int chunk,
+                                      float softcap, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0 || n_tiles <= 0) return 0;
   if (chunk < 0 || (chunk > 0 && window > 0)) return EK_ERR_ARG;
@@ -547,7 +549,7 @@ EK_EXPORT int ek_attention_prefill_tc(void* out, const void* q, int q_row_stride
 #define EK_FA(D_, CAP_)                                                                                  \
   return launch_fa<D_, CAP_>((bf16*)out, (const bf16*)q, q_row_stride, (const int4*)tiles, n_tiles,       \
                              n_tokens, k_pages, v_pages, page_rows, block_table, table_stride, n_q_heads, \
-                             n_kv_heads, scale, window, status, sink, chunk, softcap, stream)
+                             n_kv_heads, scale, window, status, sink, sinks, chunk, softcap, stream)
   if (head_dim == 64) {
     if (softcap > 0.f) EK_FA(64, true);
     EK_FA(64, false);

@@ -42,6 +42,21 @@ __global__ void scale_f32_kernel(float* x, size_t n, float scale) {
   if (i < n) x[i] *= scale;
 }
 
+// x = cap tanh(scale x / cap), four values a thread (one by one where they are not aligned, and at the end).
+__global__ void scale_cap_f32_kernel(float* x, size_t n, float scale, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float f = scale / cap;
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i + 4 <= n && ((uintptr_t)x & 15) == 0) {
+    float4 v = *reinterpret_cast<float4*>(x + i);
+    v = make_float4(cap * tanhf(v.x * f), cap * tanhf(v.y * f), cap * tanhf(v.z * f), cap * tanhf(v.w * f));
+    *reinterpret_cast<float4*>(x + i) = v;
+  } else {
+    for (size_t j = i; j < n && j < i + 4; ++j) x[j] = cap * tanhf(x[j] * f);
+  }
+}
+
 
 // y = gain * x * rsqrt(mean(x^2) + eps) for each row; x is the 32-bit stream.
 // If `add` is given, the stream first becomes stream + add (written back when
@@ -647,4 +662,12 @@ EK_EXPORT int ek_scale_f32(float* x, long long n, float scale, cudaStream_t stre
   if (n <= 0) return 0;
   return (int)ek::launch_pdl(ek::scale_f32_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x,
                              (size_t)n, scale);
+}
+
+// x[i] = cap tanh(scale x[i] / cap) for n 32-bit values (logits of a model with a soft cap on them)
+EK_EXPORT int ek_scale_cap_f32(float* x, long long n, float scale, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f) || n > (1ll << 40)) return EK_ERR_ARG;
+  return (int)ek::launch_pdl(ek::scale_cap_f32_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, stream, x,
+                             (size_t)n, scale, cap);
 }

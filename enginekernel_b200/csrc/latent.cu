@@ -18,6 +18,8 @@ namespace ek {
 
 // One block per token.  proj[t] = [dq (QR) | dkv latent (C) | key rot part (R)] in 32-bit.
 //   cq[t, :QR]   = gain_q  * dq / rms(dq)                      (type T, feeds the q up-projection)
+//                  or, without gain_q, the QR values as they are (a design whose queries - and whatever else
+//                  reads the input beside them - are plain projections); QR = 0: there is no such part
 //   page row     = [gain_kv * lat / rms(lat) | rot(r) | 0..]   (type T, D values)
 // cos/sin: [positions, rot_dims / 2] in 32-bit (any factor on them is already in the tables);
 // dimension i < rot_dims/2 of r turns with dimension i + rot_dims/2, the rest of r passes.
@@ -36,12 +38,16 @@ __global__ void latent_prepare_kernel(T* __restrict__ cq, const float* __restric
   const float* row = proj + (size_t)t * proj_stride;
   const int pos = positions[t];
 
-  float ssq = 0.f;
-  for (int i = tid; i < QR; i += blockDim.x) ssq += row[i] * row[i];
-  ssq = block_sum(ssq, scratch);
-  const float inv_q = rsqrtf(ssq / (float)QR + eps);
-  for (int i = tid; i < QR; i += blockDim.x)
-    cq[(size_t)t * QR + i] = from_f<T>(row[i] * inv_q * gain_q[i]);
+  if (gain_q != nullptr) {
+    float ssq = 0.f;
+    for (int i = tid; i < QR; i += blockDim.x) ssq += row[i] * row[i];
+    ssq = block_sum(ssq, scratch);
+    const float inv_q = rsqrtf(ssq / (float)QR + eps);
+    for (int i = tid; i < QR; i += blockDim.x)
+      cq[(size_t)t * QR + i] = from_f<T>(row[i] * inv_q * gain_q[i]);
+  } else {
+    for (int i = tid; i < QR; i += blockDim.x) cq[(size_t)t * QR + i] = from_f<T>(row[i]);
+  }
 
   if (!write_cache || pos < 0) return;            // (uniform over the block)
   const float* lat = row + QR;
@@ -189,10 +195,10 @@ static int launch_head_linear(T* out, int out_row_stride, int out_head_stride, c
       int QR, int C, int R, int D, int write_cache, cudaStream_t stream) {                            \
     using namespace ek;                                                                               \
     if (n_tokens <= 0) return 0;                                                                      \
-    if (QR <= 0 || C <= 0 || R < 0 || D < C + R || rot_dims < 0 || rot_dims > R || rot_dims % 2 ||    \
-        proj_stride < QR + C + R)                                                                     \
+    if (QR < 0 || (QR == 0 && gain_q) || (QR > 0 && !cq) || C <= 0 || R < 0 || D < C + R ||           \
+        rot_dims < 0 || rot_dims > R || rot_dims % 2 || proj_stride < QR + C + R)                     \
       return EK_ERR_ARG;                                                                              \
-    latent_prepare_kernel<T><<<n_tokens, 128, 0, stream>>>(                                           \
+    latent_prepare_kernel<T><<<n_tokens, QR > 2048 ? 512 : 128, 0, stream>>>(                         \
         (T*)cq, proj, proj_stride, gain_q, gain_kv, eps, cos_t, sin_t, rot_dims, positions,           \
         token_slot, (T*)pages, block_table, table_stride, QR, C, R, D, write_cache);                  \
     EK_RETURN_LAUNCH_STATUS();                                                                        \

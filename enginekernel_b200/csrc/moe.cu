@@ -8,7 +8,10 @@
 //             the softmax over the chosen logits alone (times scale), taken from the logits with the
 //             chosen maximum off, so that no score can vanish against an unchosen expert's.  `mode` 2: scores
 //             are sigmoids of the logits, each for itself; the weights are the chosen scores times scale,
-//             not divided by their sum.
+//             not divided by their sum.  `mode` 3: softmax scores over all experts as weights (times scale, not
+//             divided by their sum); `correction` [E] (any sign) joins the scores for the choice only.
+//             Numbers from the plan's E on name experts without weights whose output is the input itself:
+//             the plan leaves their pairs out and `combine` adds weight * input.
 //   plan      the (token, choice) pairs sorted by expert, and the row tiles of every expert's
 //             stretch, made on the device: the host never sees who chose what.
 //   expert product  out[row] = f(x[row] . W_e^T) over the tiles of the plan: FFMA with 32-bit
@@ -21,8 +24,8 @@
 //             act(gate) * up from the 32-bit sums (N counts the weight rows, the output has N / 2).
 //             `row_weight` (up form): a pair's weight multiplies its row of the product before the activation,
 //             which is the product of the weighted input; `limit` belongs to the clamped activation.
-//   combine   out[t] = sum over the token's choices, in the order they were chosen (+ add[t], the result of an
-//             expert that every token shares).
+//   combine   out[t] = sum over the token's choices, in the order they were chosen (a choice that names an
+//             expert without weights adds weight * x[t]) (+ add[t], the result of an expert that every token shares).
 #include "common.cuh"
 
 namespace ek {
@@ -42,9 +45,10 @@ constexpr int kRouteWarps = 4;
 __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
                  const float* __restrict__ logits, int n_tokens, int E, int n_groups, int keep, int top,
-                 float scale, int mode) {
-  // mode 0: softmax scores, divided by the chosen ones' sum; 1: softmax over the chosen; 2: sigmoids as they are
-  const bool among_chosen = mode != 0;          // (candidates are compared by their logits)
+                 float scale, int mode, const float* __restrict__ correction) {
+  // mode 0: softmax scores, divided by the chosen ones' sum; 1: softmax over the chosen; 2: sigmoids as they are;
+  // 3: softmax scores as they are, chosen by score + correction
+  const bool among_chosen = mode == 1 || mode == 2;     // (candidates are compared by their logits)
   extern __shared__ float route_s[];            // per warp: scores [E], candidates [E], groups [n_groups]
   pdl_launch_dependents();
   pdl_wait();
@@ -64,8 +68,11 @@ moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
   const float inv = 1.f / sum;
   // candidates: the scores; with weights among the chosen the logits themselves, so that the order of
   // two experts whose scores both round to nothing is still the order of their logits
-  const float shut = among_chosen ? -INFINITY : -2.f;
-  for (int e = lane; e < E; e += 32) { s[e] *= inv; cand[e] = among_chosen ? z[e] : s[e]; }
+  const float shut = mode != 0 ? -INFINITY : -2.f;
+  for (int e = lane; e < E; e += 32) {
+    s[e] *= inv;
+    cand[e] = among_chosen ? z[e] : correction != nullptr ? s[e] + correction[e] : s[e];
+  }
   __syncwarp();
   if (n_groups > 1 && keep < n_groups) {
     const int per = E / n_groups;
@@ -120,7 +127,7 @@ moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
       sel_weight[(size_t)t * top + k] = expf(z[sel_expert[(size_t)t * top + k]] - z0) / den * scale;
     return;
   }
-  const float f = scale / (total + 1e-20f);
+  const float f = mode == 3 ? scale : scale / (total + 1e-20f);
   for (int k = lane; k < top; k += 32) sel_weight[(size_t)t * top + k] *= f;
 }
 
@@ -418,16 +425,45 @@ moe_expert_product_tc_kernel(void* __restrict__ out_, const bf16* __restrict__ a
     }
 }
 
-// out[t, :] = sum_k pair_out[t * top + k, :], k ascending.
+// out[t, :] = sum_k pair_out[t * top + k, :], k ascending (+ add[t, :]).  A choice k whose expert number is E or more
+// (`chosen` given) has no row in pair_out: weight[t, k] * x[t, :] takes its place.  Four values a thread when `vec`.
 template <typename T>
-__global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ pair_out, int top,
-                                   int width, const T* __restrict__ add) {
+__global__ void __launch_bounds__(256)
+moe_combine_kernel(T* __restrict__ out, const float* __restrict__ pair_out, int top, int width,
+                   const T* __restrict__ add, const int* __restrict__ chosen, const float* __restrict__ weight,
+                   const T* __restrict__ x, int E, int vec) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 xv = chosen ? Vec4<T>::load(x + t * width + i) : a;
+#pragma unroll 4
+      for (int k = 0; k < top; ++k) {
+        float w = 1.f;
+        float4 v;
+        if (chosen && chosen[t * top + k] >= E) {
+          w = weight[t * top + k];
+          v = xv;
+        } else {
+          v = *reinterpret_cast<const float4*>(pair_out + (t * top + k) * width + i);
+        }
+        a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+      }
+      if (add) {
+        const float4 s = Vec4<T>::load(add + t * width + i);
+        a.x += s.x; a.y += s.y; a.z += s.z; a.w += s.w;
+      }
+      Vec4<T>::store(out + t * width + i, a);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float a = 0.f;
-    for (int k = 0; k < top; ++k) a += pair_out[(t * top + k) * width + i];
+    for (int k = 0; k < top; ++k)
+      a += chosen && chosen[t * top + k] >= E ? weight[t * top + k] * to_f<T>(x[t * width + i])
+                                              : pair_out[(t * top + k) * width + i];
     if (add) a += to_f<T>(add[t * width + i]);
     out[t * width + i] = from_f<T>(a);
   }
@@ -439,11 +475,12 @@ EK_EXPORT int ek_moe_tile_rows() { return ek::kTileRows; }
 
 EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logits, int n_tokens, int E,
                            int n_groups, int keep, int top, float scale, int mode,
-                           cudaStream_t stream) {
+                           const float* correction, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
-      top > keep * (E / n_groups) || mode < 0 || mode > 2 || (mode == 2 && keep < n_groups))
+      top > keep * (E / n_groups) || mode < 0 || mode > 3 || (mode >= 2 && keep < n_groups) ||
+      (correction && mode != 3))
     return EK_ERR_ARG;
   const size_t smem = (size_t)kRouteWarps * (2 * E + n_groups) * sizeof(float);
   if (smem > 200 * 1024) return EK_ERR_ARG;
@@ -452,7 +489,7 @@ EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logi
     if (e != cudaSuccess) return (int)e;
   }
   moe_route_kernel<<<(n_tokens + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, stream>>>(
-      sel_expert, sel_weight, logits, n_tokens, E, n_groups, keep, top, scale, mode);
+      sel_expert, sel_weight, logits, n_tokens, E, n_groups, keep, top, scale, mode, correction);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -527,9 +564,15 @@ EK_EXPORT int ek_moe_expert_down_tc(float* out, const void* a, const void* w, co
     EK_RETURN_LAUNCH_STATUS();                                                                        \
   }                                                                                                   \
   EK_EXPORT int ek_moe_combine_##SUFFIX(void* out, const float* pair_out, int n_tokens, int top,      \
-                                        int width, const void* add, cudaStream_t stream) {            \
+                                        int width, const void* add, const int* chosen,                \
+                                        const float* weight, const void* x, int E,                    \
+                                        cudaStream_t stream) {                                        \
     if (n_tokens <= 0) return 0;                                                                      \
-    ek::moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>((T*)out, pair_out, top, width, (const T*)add); \
+    if (width <= 0 || top <= 0 || (chosen && (!weight || !x))) return EK_ERR_ARG;                     \
+    const uintptr_t rows = (uintptr_t)out | (uintptr_t)add | (uintptr_t)x;                            \
+    const int vec = width % 4 == 0 && ((uintptr_t)pair_out & 15) == 0 && (rows & (4 * sizeof(T) - 1)) == 0; \
+    ek::moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>((T*)out, pair_out, top, width, (const T*)add, \
+                                                            chosen, weight, (const T*)x, E, vec);     \
     EK_RETURN_LAUNCH_STATUS();                                                                        \
   }
 

@@ -20,6 +20,9 @@
 //   ssm_out          (o + D x) silu(z), RMS norm in equal parts, weight -> activation type
 //   norm_gate_out    RMS norm over all heads together, weight, sigmoid gate -> activation type (a matrix state
 //                    whose decays are one constant per head: decay_scan with a and b the same for every token)
+//   rotate_heads     rotary positions on heads of a 32-bit projection, in place (queries and keys that enter a
+//                    matrix state rotated)
+//   head_norm_gate_out  RMS norm per head, optional weight, SiLU or sigmoid gate -> activation type
 //   xlstm_out        o / (max(|n.q|, exp(-m)) + 1e-6), RMS norm per head, weight, sigmoid gate
 // and a recurrence with a decay per CHANNEL and no matrix state (a gated linear recurrent unit):
 //   lru_gates        both gates from block-diagonal products, the decay and the gated input
@@ -894,7 +897,123 @@ norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float
   for (int i = threadIdx.x + kOutKeep * blockDim.x; i < inner; i += blockDim.x)
     y[t * inner + i] = from_f<T>(row[i] * rstd * w[i] * sigmoid_f(gate[i]));
 }
+
+// x[t, col0 + h * dim + .] rotated in place for `heads` neighbouring heads of a 32-bit row: values (i, i + rot / 2) of
+// each head turn by the angle of the token's position, values from `rot` on stay.  A block a token, a thread one
+// place in the head (`vec`: four) for every head it takes.
+constexpr int kRotatePasses = 4;     // heads a thread loads before it stores the first
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(float* x, int stride, int col0, int heads, int dim, int rot, const float* __restrict__ cos_t,
+                    const float* __restrict__ sin_t, const int* __restrict__ positions, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int pos = positions[t];
+  if (pos < 0) return;
+  float* row = x + t * stride + col0;
+  const int half = rot / 2;
+  const float* cs = cos_t + (size_t)pos * half;
+  const float* sn = sin_t + (size_t)pos * half;
+  if (vec) {
+    const int per = half / 4;                    // threads a head (at most the block's)
+    const int step = blockDim.x / per, i = (threadIdx.x % per) * 4, h0 = threadIdx.x / per;
+    if (h0 >= step) return;
+    const float4 c = *reinterpret_cast<const float4*>(cs + i), s = *reinterpret_cast<const float4*>(sn + i);
+    for (int base = h0; base < heads; base += step * kRotatePasses) {
+      float4 u[kRotatePasses], v[kRotatePasses];
+#pragma unroll
+      for (int p = 0; p < kRotatePasses; ++p) {
+        const int h = base + p * step;
+        if (h >= heads) continue;
+        u[p] = *reinterpret_cast<const float4*>(row + (size_t)h * dim + i);
+        v[p] = *reinterpret_cast<const float4*>(row + (size_t)h * dim + half + i);
+      }
+#pragma unroll
+      for (int p = 0; p < kRotatePasses; ++p) {
+        const int h = base + p * step;
+        if (h >= heads) continue;
+        const float4 a = u[p], b = v[p];
+        *reinterpret_cast<float4*>(row + (size_t)h * dim + i) =
+            make_float4(a.x * c.x - b.x * s.x, a.y * c.y - b.y * s.y, a.z * c.z - b.z * s.z, a.w * c.w - b.w * s.w);
+        *reinterpret_cast<float4*>(row + (size_t)h * dim + half + i) =
+            make_float4(b.x * c.x + a.x * s.x, b.y * c.y + a.y * s.y, b.z * c.z + a.z * s.z, b.w * c.w + a.w * s.w);
+      }
+    }
+    return;
+  }
+  for (int n = threadIdx.x; n < heads * half; n += blockDim.x) {
+    const int h = n / half, i = n % half;
+    float* p = row + (size_t)h * dim + i;
+    const float u = p[0], v = p[half], c = cs[i], s = sn[i];
+    p[0] = u * c - v * s;
+    p[half] = v * c + u * s;
+  }
+}
+
+// A warp a token and head, 8 warps a block: y[t, h, j] = o / rms(o over the head) * w[h vdim + j] (w null: 1) * act(gate)
+// with gate = proj[t, col_g + h vdim + j]; act 0: sigmoid, 1: SiLU.
+template <typename T>
+__global__ void __launch_bounds__(32 * kOutWarps)
+head_norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float* __restrict__ proj,
+                          int proj_stride, int col_g, const float* __restrict__ w, float eps, int silu,
+                          const int* __restrict__ positions, int n_tokens, int heads, int vdim, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long pair = (long long)blockIdx.x * kOutWarps + (threadIdx.x >> 5);
+  if (pair >= (long long)n_tokens * heads) return;
+  const int t = (int)(pair / heads), h = (int)(pair % heads);
+  if (positions[t] < 0) return;
+  const float* oh = o + (size_t)pair * vdim;
+  const float* gate = proj + (size_t)t * proj_stride + col_g + (size_t)h * vdim;
+  const float* wh = w ? w + (size_t)h * vdim : nullptr;
+  T* yh = y + (size_t)pair * vdim;
+  auto gated = [&](float u, float g) { return silu ? u * g * sigmoid_f(g) : u * sigmoid_f(g); };
+  float ss = 0.f;
+  constexpr int kKeep4 = 2;                      // up to 256 values a head stay in registers
+  if (vec && vdim <= 128 * kKeep4) {
+    float4 u[kKeep4], g[kKeep4];
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m) {
+      const int i = (lane + 32 * m) * 4;
+      u[m] = g[m] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < vdim) {
+        u[m] = *reinterpret_cast<const float4*>(oh + i);
+        g[m] = *reinterpret_cast<const float4*>(gate + i);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m) ss += u[m].x * u[m].x + u[m].y * u[m].y + u[m].z * u[m].z + u[m].w * u[m].w;
+    const float r = rsqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+    for (int m = 0; m < kKeep4; ++m) {
+      const int i = (lane + 32 * m) * 4;
+      if (i >= vdim) continue;
+      float4 f = make_float4(r, r, r, r);
+      if (wh) { const float4 w4 = *reinterpret_cast<const float4*>(wh + i); f.x *= w4.x; f.y *= w4.y; f.z *= w4.z; f.w *= w4.w; }
+      Vec4<T>::store(yh + i, make_float4(gated(u[m].x * f.x, g[m].x), gated(u[m].y * f.y, g[m].y),
+                                         gated(u[m].z * f.z, g[m].z), gated(u[m].w * f.w, g[m].w)));
+    }
+    return;
+  }
+  for (int i = lane; i < vdim; i += 32) ss += oh[i] * oh[i];
+  const float r = rsqrtf(warp_sum(ss) / (float)vdim + eps);
+  for (int i = lane; i < vdim; i += 32) yh[i] = from_f<T>(gated(oh[i] * r * (wh ? wh[i] : 1.f), gate[i]));
+}
 }  // namespace ek
+
+EK_EXPORT int ek_rotate_heads(float* x, int stride, int col0, int heads, int dim, int rot, const float* cos_t,
+                              const float* sin_t, const int* positions, int n_tokens, cudaStream_t stream) {
+  using namespace ek;
+  if (n_tokens <= 0 || rot == 0) return 0;
+  if (heads <= 0 || dim <= 0 || rot < 0 || rot % 2 || rot > dim || col0 < 0 || col0 + (long long)heads * dim > stride ||
+      !cos_t || !sin_t)
+    return EK_ERR_ARG;
+  const int vec = rot % 8 == 0 && rot <= 8 * 256 && dim % 4 == 0 && stride % 4 == 0 && col0 % 4 == 0 &&
+                  (((uintptr_t)x | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0;
+  return (int)launch_pdl(rotate_heads_kernel, dim3(n_tokens), dim3(256), 0, stream, x, stride, col0, heads, dim, rot,
+                         cos_t, sin_t, positions, vec);
+}
 
 #define EK_INSTANTIATE(SUFFIX, T)                                                                              \
   EK_EXPORT int ek_ssm_out_##SUFFIX(void* y, const float* o, const float* x, int x_stride, const float* proj,  \
@@ -932,6 +1051,21 @@ norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const float
     return (int)ek::launch_pdl(ek::xlstm_out_kernel<T>, dim3((unsigned)blocks), dim3(32 * ek::kOutWarps), 0,   \
                                stream, (T*)y, o, m_run, proj, proj_stride, col_g, w, eps, q_scale, positions,  \
                                n_tokens, heads, vdim);                                                         \
+  }                                                                                                            \
+  EK_EXPORT int ek_head_norm_gate_out_##SUFFIX(void* y, const float* o, const float* proj, int proj_stride,    \
+                                               int col_g, const float* w, float eps, int silu,                 \
+                                               const int* positions, int n_tokens, int heads, int vdim,        \
+                                               cudaStream_t stream) {                                          \
+    if (n_tokens <= 0) return 0;                                                                               \
+    if (heads <= 0 || vdim <= 0 || col_g < 0 || col_g + (long long)heads * vdim > proj_stride) return EK_ERR_ARG; \
+    const long long blocks = ((long long)n_tokens * heads + ek::kOutWarps - 1) / ek::kOutWarps;                \
+    if (blocks > 0x7fffffffLL) return EK_ERR_ARG;                                                              \
+    const int vec = vdim % 4 == 0 && proj_stride % 4 == 0 && col_g % 4 == 0 &&                                 \
+                    ((uintptr_t)y & (4 * sizeof(T) - 1)) == 0 &&                                               \
+                    (((uintptr_t)o | (uintptr_t)proj | (uintptr_t)w) & 15) == 0;                               \
+    return (int)ek::launch_pdl(ek::head_norm_gate_out_kernel<T>, dim3((unsigned)blocks),                       \
+                               dim3(32 * ek::kOutWarps), 0, stream, (T*)y, o, proj, proj_stride, col_g, w, eps, \
+                               silu, positions, n_tokens, heads, vdim, vec);                                   \
   }
 
 EK_INSTANTIATE(f32, float)

@@ -589,6 +589,145 @@ static int launch(void* qkv, int row_stride, const float* q_gain, const float* k
                          token_slot, cache, n_q_heads, eps, write_kv, ex);
 }
 
+// Queries and keys normed over the whole projection - all query heads of a token together, and all its key heads -
+// before they are cut into heads and rotated.  A block a token: every value times its gain waits in shared memory
+// for both root mean squares, values go straight to their pages.  Rows hold query heads from column 0, key heads
+// and value heads behind them, each `D` = the cache's head size apart; heads may be padded with zeros beyond the
+// values they have, `norm_dim` is the count a head brings to the mean.  The gains are [heads * D].
+// `vec`: four neighbouring values a thread (D % 4 == 0, rot_dim % 8 == 0, everything aligned); a thread then keeps
+// one place in the head for all heads it takes, and with it its cosines and sines.
+constexpr int kWholePasses = 4;      // heads a thread loads before it uses the first
+template <typename T>
+__global__ void __launch_bounds__(512)
+qk_whole_norm_rope_kv_kernel(T* rows, int row_stride, const float* __restrict__ q_gain,
+                             const float* __restrict__ k_gain, const float* __restrict__ cos_tab,
+                             const float* __restrict__ sin_tab, int rot_dim, const int* positions,
+                             const int* token_slot, PagedKV cache, int n_q, int norm_dim, float eps,
+                             int write_kv, int vec) {
+  extern __shared__ __align__(16) float vals[];              // [(n_q + n_kv) * D], value * gain
+  __shared__ float part_q[16], part_k[16];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int D = cache.head_dim, n_kv = cache.heads, half = rot_dim >> 1;
+  const int n_norm = write_kv ? n_q + n_kv : n_q, n_heads = write_kv ? n_q + 2 * n_kv : n_q;
+  const int pos = positions[t];
+  if (pos < 0) return;
+  T* row = rows + (size_t)t * row_stride;
+  int page = 0;
+  if (write_kv) page = cache.block_table[(size_t)token_slot[t] * cache.table_stride + pos / EK_PAGE];
+  const int per_head = vec ? D >> 2 : 1, head_step = (int)blockDim.x / per_head;
+  const int head0 = tid / per_head, j = (tid % per_head) * 4;
+  const bool mine = vec && head0 < head_step;
+  float sq = 0.f, sk = 0.f;
+  if (mine) {
+    for (int base = head0; base < n_heads; base += head_step * kWholePasses) {
+      float4 v[kWholePasses];
+#pragma unroll
+      for (int p = 0; p < kWholePasses; ++p) {
+        const int head = base + p * head_step;
+        if (head < n_heads) v[p] = Vec4<T>::load(row + (size_t)head * D + j);
+      }
+#pragma unroll
+      for (int p = 0; p < kWholePasses; ++p) {
+        const int head = base + p * head_step;
+        if (head >= n_heads) continue;
+        if (head >= n_norm) {                    // a value head: as projected
+          Vec4<T>::store((T*)cache.v + page_offset(cache, page, head - n_norm, pos) + j, v[p]);
+          continue;
+        }
+        const float ss = v[p].x * v[p].x + v[p].y * v[p].y + v[p].z * v[p].z + v[p].w * v[p].w;
+        if (head < n_q) sq += ss; else sk += ss;
+        const float4 g = *reinterpret_cast<const float4*>((head < n_q ? q_gain + (size_t)head * D
+                                                                      : k_gain + (size_t)(head - n_q) * D) + j);
+        *reinterpret_cast<float4*>(vals + (size_t)head * D + j) =
+            make_float4(v[p].x * g.x, v[p].y * g.y, v[p].z * g.z, v[p].w * g.w);
+      }
+    }
+  } else if (!vec) {
+    for (int i = tid; i < n_heads * D; i += blockDim.x) {
+      const float v = to_f<T>(row[i]);
+      if (i >= n_norm * D) {
+        ((T*)cache.v)[page_offset(cache, page, i / D - n_norm, pos) + i % D] = row[i];
+      } else if (i < n_q * D) {
+        sq += v * v;
+        vals[i] = v * q_gain[i];
+      } else {
+        sk += v * v;
+        vals[i] = v * k_gain[i - n_q * D];
+      }
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { part_q[warp] = sq; part_k[warp] = sk; }
+  __syncthreads();
+  const int n_warps = (int)blockDim.x >> 5;
+  sq = sk = 0.f;
+  for (int w = 0; w < n_warps; ++w) { sq += part_q[w]; sk += part_k[w]; }
+  const float rq = rsqrtf(sq / (float)(n_q * norm_dim) + eps), rk = rsqrtf(sk / (float)(n_kv * norm_dim) + eps);
+  const float* cs = cos_tab + (size_t)pos * half;
+  const float* sn = sin_tab + (size_t)pos * half;
+  if (mine) {
+    float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
+    int partner = j;
+    if (j < rot_dim) {
+      const int a = j < half ? j : j - half;
+      c = *reinterpret_cast<const float4*>(cs + a);
+      s = *reinterpret_cast<const float4*>(sn + a);
+      if (j < half) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+      partner = j < half ? j + half : j - half;
+    }
+    for (int head = head0; head < n_norm; head += head_step) {
+      const float r = head < n_q ? rq : rk;
+      const float4 x = *reinterpret_cast<const float4*>(vals + (size_t)head * D + j);
+      const float4 y = *reinterpret_cast<const float4*>(vals + (size_t)head * D + partner);
+      T* dst = head < n_q ? row + (size_t)head * D + j
+                          : (T*)cache.k + page_offset(cache, page, head - n_q, pos) + j;
+      Vec4<T>::store(dst, make_float4((x.x * c.x + y.x * s.x) * r, (x.y * c.y + y.y * s.y) * r,
+                                      (x.z * c.z + y.z * s.z) * r, (x.w * c.w + y.w * s.w) * r));
+    }
+  } else if (!vec) {
+    for (int i = tid; i < n_norm * D; i += blockDim.x) {
+      const int head = i / D, d = i % D;
+      float y = vals[i];
+      if (d < half) y = y * cs[d] - vals[i + half] * sn[d];
+      else if (d < rot_dim) y = y * cs[d - half] + vals[i - half] * sn[d - half];
+      y *= head < n_q ? rq : rk;
+      if (head < n_q) row[i] = from_f<T>(y);
+      else ((T*)cache.k)[page_offset(cache, page, head - n_q, pos) + d] = from_f<T>(y);
+    }
+  }
+}
+
+template <typename T>
+static int launch_whole(void* rows, int row_stride, const float* q_gain, const float* k_gain, const float* cos_tab,
+                        const float* sin_tab, int rot_dim, const int* positions, const int* token_slot,
+                        void* k_pages, void* v_pages, const int* block_table, int table_stride, int n_tokens,
+                        int n_q_heads, int n_kv_heads, int head_dim, int norm_dim, float eps, int write_kv,
+                        cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (head_dim <= 0 || head_dim > EK_MAX_HEAD_DIM || rot_dim < 0 || rot_dim % 2 || rot_dim > head_dim ||
+      norm_dim <= 0 || norm_dim > head_dim || n_q_heads <= 0 || n_kv_heads <= 0 || !q_gain || (write_kv && !k_gain))
+    return EK_ERR_ARG;
+  const long long values = (long long)(n_q_heads + (write_kv ? n_kv_heads : 0)) * head_dim;
+  if (values > 50 * 1024) return EK_ERR_ARG;
+  const size_t smem = (size_t)values * sizeof(float);
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(qk_whole_norm_rope_kv_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  const uintptr_t wide = (uintptr_t)q_gain | (uintptr_t)k_gain | (rot_dim ? (uintptr_t)cos_tab | (uintptr_t)sin_tab : 0);
+  const uintptr_t narrow = (uintptr_t)rows | (uintptr_t)k_pages | (uintptr_t)v_pages;
+  const int vec = head_dim % 4 == 0 && rot_dim % 8 == 0 && row_stride % 4 == 0 && (wide & 15) == 0 &&
+                  (narrow & (4 * sizeof(T) - 1)) == 0;
+  PagedKV cache{k_pages, v_pages, block_table, table_stride, n_kv_heads, head_dim};
+  return (int)launch_pdl(qk_whole_norm_rope_kv_kernel<T>, dim3(n_tokens), dim3(values > 4096 ? 512 : 256), smem, stream,
+                         (T*)rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, rot_dim, positions, token_slot,
+                         cache, n_q_heads, norm_dim, eps, write_kv, vec);
+}
+
 }  // namespace ek
 
 #define EK_INSTANTIATE(SUFFIX, T)                                                              \
@@ -656,6 +795,19 @@ static int launch(void* qkv, int row_stride, const float* q_gain, const float* k
                            (T*)rows, row_stride, k_col, v_col, cos_tab, sin_tab, rot_dim,      \
                            positions, token_slot, cache, n_q_heads, norm_dim, eps, unit,       \
                            write_kv);                                                          \
+  }                                                                                            \
+  /* The gained norm of queries and of keys over the whole projection (gains [heads * D]),    */ \
+  /* then the rotation; heads may be padded with zeros beyond norm_dim values.                */ \
+  EK_EXPORT int ek_qk_whole_norm_kv_##SUFFIX(                                                   \
+      void* rows, int row_stride, const float* q_gain, const float* k_gain,                    \
+      const float* cos_tab, const float* sin_tab, int rot_dim, const int* positions,           \
+      const int* token_slot, void* k_pages, void* v_pages, const int* block_table,             \
+      int table_stride, int n_tokens, int n_q_heads, int n_kv_heads, int head_dim,             \
+      int norm_dim, float eps, int write_kv, cudaStream_t stream) {                            \
+    return ek::launch_whole<T>(rows, row_stride, q_gain, k_gain, cos_tab, sin_tab, rot_dim,    \
+                               positions, token_slot, k_pages, v_pages, block_table,           \
+                               table_stride, n_tokens, n_q_heads, n_kv_heads, head_dim,        \
+                               norm_dim, eps, write_kv, stream);                               \
   }
 
 EK_INSTANTIATE(f32, float)

@@ -220,7 +220,9 @@ class DecoderModel:
         h = self.final_norm.forward(stream, ctx, add=pending, rows=rows, n_rows=n_rows,
                                     write_back=False)
         out = linear(h, self.lm_head, ctx, "logits", n_rows=n_rows, out_dtype=torch.float32)
-        if self.spec.logit_multiplier != 1.0:
+        if self.spec.logit_softcap is not None:
+            kernels.scale_cap_(out, self.spec.logit_multiplier, self.spec.logit_softcap)
+        elif self.spec.logit_multiplier != 1.0:
             kernels.scale_(out, self.spec.logit_multiplier)
         return out
 

@@ -20,6 +20,7 @@ from .lib import Function, KernelError, count_extra_launches
 PAGE = 64                 # tokens per cache page; must equal EK_PAGE in csrc/common.cuh
 MAX_HEAD_DIM = 256        # of the 16-bit attention kernels
 PREPARE_MAX_HEAD_DIM = 512      # of the kernels that norm, rotate and store heads; equals EK_MAX_HEAD_DIM in csrc/common.cuh
+WHOLE_NORM_MAX_VALUES = 50 * 1024     # query and key values of a token that qk_whole_norm_kv keeps in shared memory
 GENERIC_MAX_HEAD_DIM = 1024     # the general attention kernel alone takes head sizes up to here
 
 _SUFFIX = {torch.float32: "f32", torch.bfloat16: "bf16"}
@@ -94,6 +95,7 @@ def _per_dtype(module, name, argtypes):
 # ------------------------------------------------------------------ elementwise
 _embed = _per_dtype("elementwise", "ek_embed", [_P, _P, _P, c_int, c_int, c_int, c_float, _P, _P, c_int, c_int, _P])
 _scale_f32 = Function("elementwise", "ek_scale_f32", [_P, c_longlong, c_float, _P])
+_scale_cap_f32 = Function("elementwise", "ek_scale_cap_f32", [_P, c_longlong, c_float, c_float, _P])
 _rmsnorm = _per_dtype("elementwise", "ek_rmsnorm",
                       [_P, _P, _P, _P, _P, c_float, c_int, c_int, c_int, _P])
 _add_residual = _per_dtype("elementwise", "ek_add_residual", [_P, _P, c_longlong, _P])
@@ -133,6 +135,16 @@ def scale_(x, scale, n=None):
     if lib.recording():
         lib.annotate(bytes=8 * count)
     _scale_f32(_ptr(x), count, float(scale), _stream())
+
+
+def scale_cap_(x, scale, cap, n=None):
+    """x <- cap tanh(scale x / cap) in place (32-bit values; the first ``n`` of them)."""
+    _need_cuda(x)
+    _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "scale_cap_: contiguous 32-bit values, a positive cap")
+    count = x.numel() if n is None else n
+    if lib.recording():
+        lib.annotate(bytes=8 * count)
+    _scale_cap_f32(_ptr(x), count, float(scale), float(cap), _stream())
 
 
 def rmsnorm(y, resid, gain, eps, add=None, rows=None, n_rows=None, write_back=True):
@@ -514,6 +526,40 @@ def qk_norm_rope_kv(qkv, n_tokens, q_gain, k_gain, cos, sin, rot_dim, positions,
                         head_dim, float(eps), 1 if write_kv else 0, _stream())
 
 
+_whole_norm_kv = _per_dtype("rope_kv", "ek_qk_whole_norm_kv",
+                            [_P, c_int, _P, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
+                             c_int, c_float, c_int, _P])
+
+
+def qk_whole_norm_kv(rows, n_tokens, q_gain, k_gain, cos, sin, rot_dim, positions, token_slot, k_pages, v_pages,
+                     block_table, n_q_heads, n_kv_heads, head_dim, eps, norm_dim=None, write_kv=True):
+    """Queries and keys normed over the whole projection before they are cut into heads: all query heads of a
+    token share one root mean square, all its key heads another (gains [heads * D], 32-bit); then the rotation.
+    ``rows`` [T, .] holds query, key and value heads ``head_dim`` apart (keys and values are read only when
+    ``write_kv``); queries stay in place, keys and values go to the pages.  ``norm_dim``: values a head really has,
+    when heads are padded with zeros."""
+    _need_cuda(rows, q_gain, k_gain, cos, sin, positions, token_slot, k_pages, v_pages, block_table)
+    check_head_dim(head_dim)
+    heads = n_q_heads + (2 * n_kv_heads if write_kv else 0)
+    _need((n_q_heads + n_kv_heads) * head_dim <= WHOLE_NORM_MAX_VALUES,
+          f"qk_whole_norm_kv: query and key heads of a token hold at most {WHOLE_NORM_MAX_VALUES} values together")
+    _need(rows.stride(-1) == 1 and rows.shape[-1] >= heads * head_dim, "qk_whole_norm_kv: row width")
+    _need(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous()
+          and cos.shape[-1] * 2 == rot_dim, "qk_whole_norm_kv: 32-bit tables of rot_dim/2 columns")
+    _need(k_pages.dtype == rows.dtype and v_pages.dtype == rows.dtype, "qk_whole_norm_kv: cache dtype")
+    _need(block_table.dtype == torch.int32 and positions.dtype == torch.int32
+          and token_slot.dtype == torch.int32, "qk_whole_norm_kv: int32 indices")
+    for g, n in ((q_gain, n_q_heads),) + (((k_gain, n_kv_heads),) if write_kv else ()):
+        _need(g is not None and g.dtype == torch.float32 and g.is_contiguous() and g.numel() == n * head_dim,
+              "qk_whole_norm_kv: gains are 32-bit [heads * D]")
+    if lib.recording():
+        lib.annotate(bytes=n_tokens * head_dim * rows.element_size() * (2 * n_q_heads + (4 * n_kv_heads if write_kv else 0)))
+    _whole_norm_kv[rows.dtype](_ptr(rows), rows.stride(0), _ptr(q_gain), _ptr(k_gain), _ptr(cos), _ptr(sin), rot_dim,
+                               _ptr(positions), _ptr(token_slot), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
+                               block_table.stride(0), n_tokens, n_q_heads, n_kv_heads, head_dim,
+                               int(norm_dim or head_dim), float(eps), 1 if write_kv else 0, _stream())
+
+
 _rope_unit_kv = _per_dtype("rope_kv", "ek_qk_rope_unit_kv",
                            [_P, c_int, c_int, c_int, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int,
                             c_int, c_int, c_int, c_int, c_float, c_int, c_int, _P])
@@ -573,7 +619,7 @@ def attention_generic(out, q, n_tokens, positions, token_slot, k_pages, v_pages,
     """out[t, h*D:(h+1)*D] = softmax(scale q.K^T) V over the keys token t may see.  ``sink``: the
     score of one more key without a value that every query sees - exp(sink) is added to the
     softmax denominator (the same in every attention kernel below).  ``sinks`` [NQ] (32-bit):
-    one such score per query head instead (here and in the two mma.sync kernels).
+    one such score per query head instead (in every attention kernel).
 
     ``q`` is any tensor whose row t starts with the NQ*D query values (the fused q/k/v
     rows qualify).  With ``n_splits`` > 1 the keys are cut every ``keys_per_split`` and
@@ -733,7 +779,7 @@ def attention_decode_bf16(out, q, n_tokens, positions, token_slot, k_pages, v_pa
 
 _attn_decode_tma = Function("attention_decode_tma", "ek_attention_decode_tma",
                             [_P, _P, c_int, _P, _P, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int,
-                             c_float, c_int, c_int, _P, c_float, c_int, c_float, _P])
+                             c_float, c_int, c_int, _P, c_float, _P, c_int, c_float, _P])
 _attn_decode_tma_max = Function("attention_decode_tma", "ek_attention_decode_tma_max_splits", [c_int],
                                 check_status=False)
 DECODE_TMA_PORTABLE_SPLITS = 8
@@ -757,7 +803,7 @@ def attention_decode_tma_supported(dtype, head_dim, n_q_heads, n_kv_heads):
 
 def attention_decode_tma(out, q, n_tokens, positions, token_slot, k_pages, v_pages, block_table,
                          n_q_heads, n_kv_heads, head_dim, scale, window=None, n_splits=1, sink=None, chunk=None,
-                         softcap=None):
+                         softcap=None, sinks=None):
     """One new token per sequence (bfloat16, head size 64 or 128, at most 16 heads a group): the
     cache pages come by TMA, started before the kernel ahead has finished; ``n_splits`` (1 to 8)
     blocks (16 where :func:`decode_tma_max_splits` says so) share a token's pages and merge inside
@@ -783,8 +829,8 @@ def attention_decode_tma(out, q, n_tokens, positions, token_slot, k_pages, v_pag
     _attn_decode_tma(_ptr(out), _ptr(q), q.stride(0), _ptr(positions), _ptr(token_slot),
                      _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table),
                      block_table.stride(0), n_tokens, n_q_heads, n_kv_heads, head_dim, float(scale),
-                     int(window or 0), n_splits, _ptr(tc_status(q.device)), _sink(sink), int(chunk or 0),
-                     float(softcap or 0.0), _stream())
+                     int(window or 0), n_splits, _ptr(tc_status(q.device)), _sink(sink),
+                     _sinks(sinks, n_q_heads), int(chunk or 0), float(softcap or 0.0), _stream())
 
 
 _attn_prefill_bf16 = Function("attention_prefill_bf16", "ek_attention_prefill_bf16",
@@ -823,7 +869,7 @@ def attention_prefill_bf16(out, q, n_tokens, positions, token_slot, cu_seqlens, 
 
 _attn_prefill_tc = Function("attention_prefill_tc", "ek_attention_prefill_tc",
                             [_P, _P, c_int, _P, c_int, c_int, _P, _P, c_int, _P, c_int, c_int,
-                             c_int, c_int, c_float, c_int, _P, c_float, c_int, c_float, _P])
+                             c_int, c_int, c_float, c_int, _P, c_float, _P, c_int, c_float, _P])
 _attn_prefill_tiles = Function("attention_prefill_tc", "ek_attention_prefill_tiles",
                                [_P, c_int, _P, _P, _P, c_int, c_int, c_int, _P])
 _attn_prefill_cross = Function("attention_prefill_bf16", "ek_attention_prefill_cross_bf16",
@@ -893,7 +939,7 @@ def attention_prefill_tiles(tiles, n_tokens, positions, token_slot, cu_seqlens, 
 
 def attention_prefill_tc(out, q, n_tokens, positions, token_slot, cu_seqlens, n_seqs, k_pages,
                          v_pages, block_table, n_q_heads, n_kv_heads, head_dim, scale, window=None,
-                         tiles=None, n_tiles=0, sink=None, chunk=None, softcap=None):
+                         tiles=None, n_tiles=0, sink=None, chunk=None, softcap=None, sinks=None):
     """:func:`attention_prefill_bf16` on tcgen05 tensor cores (head sizes 64 and 128, groups
     that divide 128): TMA-fed pages, scores and P.V in TMEM.  ``tiles`` / ``n_tiles``: the table
     :func:`attention_prefill_tiles` made for this step (made once, before the step's first
@@ -920,7 +966,8 @@ def attention_prefill_tc(out, q, n_tokens, positions, token_slot, cu_seqlens, n_
     _attn_prefill_tc(_ptr(out), _ptr(q), q.stride(0), _ptr(tiles), n_tiles, n_tokens, _ptr(k_pages),
                      _ptr(v_pages), k_pages.shape[0], _ptr(block_table), block_table.stride(0), n_q_heads,
                      n_kv_heads, head_dim, float(scale), int(window or 0),
-                     _ptr(tc_status(q.device)), _sink(sink), int(chunk or 0), float(softcap or 0.0), _stream())
+                     _ptr(tc_status(q.device)), _sink(sink), _sinks(sinks, n_q_heads), int(chunk or 0),
+                     float(softcap or 0.0), _stream())
 
 
 # ------------------------------------------------------------------ matrix products
@@ -1433,25 +1480,28 @@ _head_linear = _per_dtype("latent", "ek_head_linear",
 
 def latent_prepare(cq, proj, n_tokens, gain_q, gain_kv, eps, cos, sin, rot_dims, positions, token_slot,
                    pages, block_table, q_rank, kv_rank, rot_dim, write_cache=True):
-    """``proj`` [T, q_rank + kv_rank + rot_dim] (32-bit): cq = gain_q * rms-normed first part (activation
+    """``proj`` [T, >= q_rank + kv_rank + rot_dim] (32-bit): cq = gain_q * rms-normed first part (activation
     type); the token's cache row (``pages`` [page, 1, PAGE, D], D >= kv_rank + rot_dim) becomes
-    [gain_kv * rms-normed latent | rotated key part | zeros]."""
+    [gain_kv * rms-normed latent | rotated key part | zeros].  ``gain_q`` None: the first ``q_rank`` values go
+    to ``cq`` as they are (plain projections that shared the product); ``q_rank`` 0 and ``cq`` None: there are none."""
     _need_cuda(cq, proj, gain_q, gain_kv, cos, sin, positions, token_slot, pages, block_table)
     _need(proj.dtype == torch.float32 and proj.stride(-1) == 1, "latent_prepare: 32-bit projections")
-    _need(cq.dtype == pages.dtype and cq.is_contiguous() and cq.shape[-1] == q_rank, "latent_prepare: cq [T, q_rank]")
+    _need((cq is None and q_rank == 0 and gain_q is None)
+          or (cq is not None and cq.dtype == pages.dtype and cq.is_contiguous() and cq.shape[-1] == q_rank),
+          "latent_prepare: cq [T, q_rank]")
     _need(pages.is_contiguous() and pages.dim() == 4 and pages.shape[1] == 1 and pages.shape[2] == PAGE,
           "latent_prepare: pages [page, 1, PAGE, D]")
-    _need(gain_q.dtype == gain_kv.dtype == torch.float32 and gain_q.numel() == q_rank
-          and gain_kv.numel() == kv_rank, "latent_prepare: 32-bit gains")
+    _need((gain_q is None or (gain_q.dtype == torch.float32 and gain_q.numel() == q_rank))
+          and gain_kv.dtype == torch.float32 and gain_kv.numel() == kv_rank, "latent_prepare: 32-bit gains")
     _need(rot_dims == 0 or (cos.dtype == torch.float32 and cos.shape[-1] == rot_dims // 2 and cos.is_contiguous()
                             and sin.is_contiguous()), "latent_prepare: cos/sin [positions, rot_dims / 2]")
     d = pages.shape[-1]
     if lib.recording():
-        lib.annotate(bytes=n_tokens * (4 * (q_rank + kv_rank + rot_dim) + cq.element_size() * (q_rank + d)))
-    _latent_prepare[cq.dtype](_ptr(cq), _ptr(proj), proj.stride(0), _ptr(gain_q), _ptr(gain_kv), float(eps),
-                              _ptr(cos), _ptr(sin), rot_dims, _ptr(positions), _ptr(token_slot), _ptr(pages),
-                              _ptr(block_table), block_table.stride(0), n_tokens, q_rank, kv_rank, rot_dim, d,
-                              1 if write_cache else 0, _stream())
+        lib.annotate(bytes=n_tokens * (4 * (q_rank + kv_rank + rot_dim) + pages.element_size() * (q_rank + d)))
+    _latent_prepare[pages.dtype](_ptr(cq), _ptr(proj), proj.stride(0), _ptr(gain_q), _ptr(gain_kv), float(eps),
+                                 _ptr(cos), _ptr(sin), rot_dims, _ptr(positions), _ptr(token_slot), _ptr(pages),
+                                 _ptr(block_table), block_table.stride(0), n_tokens, q_rank, kv_rank, rot_dim, d,
+                                 1 if write_cache else 0, _stream())
 
 
 HEAD_LINEAR_LIBRARY_ROWS = 64     # bfloat16 products per head of more rows than this go to the library
@@ -1605,6 +1655,10 @@ _ssm_out = _per_dtype("recurrent", "ek_ssm_out",
                       [_P, _P, _P, c_int, _P, c_int, c_int, _P, _P, c_float, _P, c_int, c_int, c_int, c_int, _P])
 _xlstm_out = _per_dtype("recurrent", "ek_xlstm_out",
                         [_P, _P, _P, _P, c_int, c_int, _P, c_float, c_float, _P, c_int, c_int, c_int, _P])
+_rotate_heads = Function("recurrent", "ek_rotate_heads",
+                         [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P])
+_head_norm_gate_out = _per_dtype("recurrent", "ek_head_norm_gate_out",
+                                 [_P, _P, _P, c_int, c_int, _P, c_float, c_int, _P, c_int, c_int, c_int, _P])
 DECAY_SCAN_MAX_KEY_DIM = 256
 
 
@@ -1788,6 +1842,38 @@ def norm_gate_out(y, o, proj, col_g, w, eps, positions, n_tokens):
                             n_tokens, inner, _stream())
 
 
+def rotate_heads(x, col0, heads, dim, rot_dims, cos, sin, positions, n_tokens):
+    """In place on ``x`` [T, .] (32-bit): ``heads`` heads of ``dim`` values from column ``col0``, the first
+    ``rot_dims`` of each turned (value i with value i + rot_dims / 2) by the token's angles."""
+    _need_cuda(x, cos, sin, positions)
+    _need_f32("rotate_heads", x, cos, sin)
+    _need(col0 + heads * dim <= x.shape[-1] and positions.dtype == torch.int32, "rotate_heads: heads within the rows")
+    _need(rot_dims == 0 or (cos.is_contiguous() and sin.is_contiguous() and cos.shape[-1] * 2 == rot_dims),
+          "rotate_heads: cos/sin [positions, rot_dims / 2]")
+    if rot_dims == 0:
+        return
+    if lib.recording():
+        lib.annotate(bytes=8 * n_tokens * heads * rot_dims)
+    _rotate_heads(_ptr(x), x.stride(0), col0, heads, dim, rot_dims, _ptr(cos), _ptr(sin), _ptr(positions), n_tokens,
+                  _stream())
+
+
+def head_norm_gate_out(y, o, proj, col_g, w, eps, positions, n_tokens, heads, vdim, gate_activation="sigmoid"):
+    """y = o / rms(o) per head * w * act(proj[., col_g + c]) in the activation type; ``w`` [heads * vdim] or None (no
+    weight), act ``"sigmoid"`` or ``"silu"``."""
+    _need_cuda(y, o, proj, w, positions)
+    _need_f32("head_norm_gate_out", o, proj, w)
+    _need(gate_activation in ("sigmoid", "silu"), "head_norm_gate_out: the gate takes a sigmoid or SiLU")
+    _need(y.is_contiguous() and o.is_contiguous() and y.shape[-1] == o.shape[-1] == heads * vdim
+          and (w is None or w.numel() == heads * vdim) and col_g + heads * vdim <= proj.shape[-1],
+          "head_norm_gate_out: y, o, w of one width, the gate within the rows")
+    if lib.recording():
+        lib.annotate(bytes=n_tokens * heads * vdim * (8 + y.element_size()))
+    _head_norm_gate_out[y.dtype](_ptr(y), _ptr(o), _ptr(proj), proj.stride(0), col_g, _ptr(w), float(eps),
+                                 1 if gate_activation == "silu" else 0, _ptr(positions), n_tokens, heads, vdim,
+                                 _stream())
+
+
 def xlstm_out(y, o, m_run, proj, col_g, w, eps, q_scale, positions, n_tokens, heads, vdim):
     """``o`` [T, heads * (vdim + 1)] from the scan with n . q in each head's last column, both still to
     be multiplied by ``q_scale``: u = o q_scale / (max(|n . q| q_scale, exp(-m)) + 1e-6); y = u / rms(u)
@@ -1803,12 +1889,12 @@ def xlstm_out(y, o, m_run, proj, col_g, w, eps, q_scale, positions, n_tokens, he
 
 
 # ------------------------------------------------------------------ routed experts
-_moe_route = Function("moe", "ek_moe_route", [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P])
+_moe_route = Function("moe", "ek_moe_route", [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P])
 _moe_plan = Function("moe", "ek_moe_plan", [_P, _P, _P, _P, c_int, c_int, _P])
 _moe_up = _per_dtype("moe", "ek_moe_expert_up",
                      [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
 _moe_down = _per_dtype("moe", "ek_moe_expert_down", [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P])
-_moe_combine = _per_dtype("moe", "ek_moe_combine", [_P, _P, c_int, c_int, c_int, _P, _P])
+_moe_combine = _per_dtype("moe", "ek_moe_combine", [_P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, _P])
 _moe_up_tc = Function("moe", "ek_moe_expert_up_tc",
                       [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
 _moe_down_tc = Function("moe", "ek_moe_expert_down_tc", [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P])
@@ -1819,7 +1905,7 @@ def _moe_on_tensor_cores(a, w) -> bool:
     return (a.dtype == torch.bfloat16 and w.shape[-1] % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 MOE_TILE_ROWS = 64          # must equal kTileRows in csrc/moe.cu
 EXPERT_ACTIVATIONS = {"none": 0, "relu2": 1, "silu": 2, "gelu_tanh": 3, "clamped": 4}
-ROUTE_WEIGHTS = {"scores_of_chosen": 0, "softmax_of_chosen": 1, "sigmoid": 2}
+ROUTE_WEIGHTS = {"scores_of_chosen": 0, "softmax_of_chosen": 1, "sigmoid": 2, "softmax": 3}
 
 
 def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
@@ -1827,17 +1913,22 @@ def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
     return -(-n_pairs // MOE_TILE_ROWS) + min(n_experts, n_pairs)
 
 
-def moe_route(sel_expert, sel_weight, logits, n_tokens, n_groups, keep, top, scale, weights="scores_of_chosen"):
+def moe_route(sel_expert, sel_weight, logits, n_tokens, n_groups, keep, top, scale, weights="scores_of_chosen",
+              correction=None):
     """Router: ``logits`` [T, E] 32-bit -> the ``top`` chosen experts and their weights per token, times ``scale``.
     ``weights``: ``"scores_of_chosen"``, the chosen scores of the softmax over all experts, divided by their sum;
     ``"softmax_of_chosen"``, the softmax over the chosen logits alone; ``"sigmoid"``, the chosen logits' sigmoids
-    as they are (all groups kept)."""
-    _need_cuda(sel_expert, sel_weight, logits)
+    as they are (all groups kept); ``"softmax"``, the chosen scores of the softmax over all experts as they are (all
+    groups kept), where ``correction`` [E] (32-bit) joins the scores for the choice only."""
+    _need_cuda(sel_expert, sel_weight, logits, correction)
+    _need(correction is None or (weights == "softmax" and correction.dtype == torch.float32 and correction.is_contiguous()
+                                 and correction.numel() == logits.shape[-1]),
+          "moe_route: a 32-bit correction per expert goes with the weights 'softmax'")
     _need(weights in ROUTE_WEIGHTS, f"moe_route: no weights {weights!r}")
     _need(logits.dtype == torch.float32 and logits.is_contiguous() and sel_expert.dtype == torch.int32
           and sel_weight.dtype == torch.float32, "moe_route: 32-bit logits and weights, int32 choices")
     _moe_route(_ptr(sel_expert), _ptr(sel_weight), _ptr(logits), n_tokens, logits.shape[-1], n_groups, keep,
-               top, float(scale), ROUTE_WEIGHTS[weights], _stream())
+               top, float(scale), ROUTE_WEIGHTS[weights], _ptr(correction), _stream())
 
 
 def moe_plan(sorted_pair, tiles, n_tiles, sel_expert, n_pairs, n_experts):
@@ -1881,15 +1972,24 @@ def moe_expert_down(pair_out, a, w, tiles, n_tiles, sorted_pair, pair_weight, n_
        _ptr(pair_weight), moe_max_tiles(n_pairs, e), n, k, _stream())
 
 
-def moe_combine(out, pair_out, n_tokens, top, add=None):
-    """out[t] = sum over the token's ``top`` pairs (+ add[t], in out's type)."""
+def moe_combine(out, pair_out, n_tokens, top, add=None, identity=None):
+    """out[t] = sum over the token's ``top`` pairs (+ add[t], in out's type).  ``identity=(chosen, weight, x, E)``:
+    a pair whose expert number is E or more has no row in ``pair_out``; weight * x[t] takes its place (``x`` rows in
+    out's type)."""
     _need_cuda(out, pair_out, add)
     width = out.shape[-1]
     _need(add is None or (add.dtype == out.dtype and add.is_contiguous() and add.shape[-1] == width),
           "moe_combine: what is added has out's type and width")
+    chosen, weight, x, e = identity if identity is not None else (None, None, None, 0)
+    _need_cuda(chosen, weight, x)
+    _need(identity is None or (x.dtype == out.dtype and x.is_contiguous() and x.shape[-1] == width
+                               and chosen.dtype == torch.int32 and weight.dtype == torch.float32
+                               and chosen.is_contiguous() and weight.is_contiguous()),
+          "moe_combine: identity experts take the input's rows in out's type, choices and 32-bit weights")
     if lib.recording():
-        lib.annotate(bytes=n_tokens * width * (4 * top + out.element_size() * (1 if add is None else 2)))
-    _moe_combine[out.dtype](_ptr(out), _ptr(pair_out), n_tokens, top, width, _ptr(add), _stream())
+        lib.annotate(bytes=n_tokens * width * (4 * top + out.element_size() * (1 + (add is not None) + (x is not None))))
+    _moe_combine[out.dtype](_ptr(out), _ptr(pair_out), n_tokens, top, width, _ptr(add), _ptr(chosen), _ptr(weight),
+                            _ptr(x), e, _stream())
 
 
 def build_all():

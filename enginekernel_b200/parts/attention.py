@@ -45,6 +45,9 @@ Optional parameters, all off by default, for designs that differ there:
 ``softcap``            a score s becomes softcap * tanh(s / softcap) before the softmax.
 ``pairing``            ``"neighbours"``: the rotation turns values (2i, 2i + 1) of a head instead of (i, i + rot/2);
                        the rows of the query and key projections are reordered once at load.
+``qk_norm_over``       ``"projection"``: the gained norm takes one mean over all query heads of a token and one over
+                       all its key heads (``q_norm`` [NH*D], ``k_norm`` [NKV*D]) instead of one per head.
+``sinks``              True: a learned sink score per query head (tensor ``sink`` [NH]) instead of one constant.
 ``value_dim``, ``unit_norm_after_rotation``, ``keep_first`` and ``head_gate`` send the layer down one path: a single
 product for everything that reads the input, a prepare kernel that knows padded heads, and the ``mma.sync`` or the
 general attention kernel.  The others ride on the ordinary path.
@@ -81,9 +84,12 @@ class Attention(Mixer):
             out.append(TensorSpec(w["gate"], (nh, h)))
         out.append(TensorSpec(w["o"], (h, nh * e)))
         if p.get("qk_norm_eps") is not None:
-            out.append(TensorSpec(w["q_norm"], (d,), "gain"))
+            whole = p.get("qk_norm_over", "head") == "projection"
+            out.append(TensorSpec(w["q_norm"], (nh * d if whole else d,), "gain"))
             if p.get("kv_projection", True):     # (else the keys it reads were normed by the run that stored them)
-                out.append(TensorSpec(w["k_norm"], (d,), "gain"))
+                out.append(TensorSpec(w["k_norm"], (nkv * d if whole else d,), "gain"))
+        if p.get("sinks"):
+            out.append(TensorSpec(w["sink"], (nh,)))
         sizes = {"q": nh * d, "k": nkv * d, "v": nkv * e, "o": h}
         for which in p.get("bias") or ():
             if p.get("kv_projection", True) or which in ("q", "o"):
@@ -115,12 +121,22 @@ class Attention(Mixer):
         self.values_from_keys = spec.params.get("values", "projection") == "keys"
         self.query_temperature = spec.params.get("query_temperature")
         self.sink = spec.params.get("sink")
+        self.has_sinks = bool(spec.params.get("sinks"))
+        if self.has_sinks and self.sink is not None:
+            raise ValueError("attention: one sink score for all heads or one per head, not both")
+        if spec.params.get("qk_norm_over", "head") not in ("head", "projection"):
+            raise ValueError("attention: the norm of queries and keys is over a 'head' or the 'projection'")
+        self.whole_norm = spec.params.get("qk_norm_over", "head") == "projection"
         if spec.params.get("values", "projection") not in ("projection", "keys"):
             raise ValueError("attention: values are 'projection' or 'keys'")
         if any(b not in ("q", "k", "v") for b in self.biased) or (self.values_from_keys and "v" in self.biased):
             raise ValueError("attention: bias names q, k, v (v only with a value projection)")
         if self.query_temperature is not None and int(self.query_temperature[1]) < 1:
             raise ValueError("attention: the query temperature steps every >= 1 positions")
+        if self.whole_norm and (self.qk_norm_eps is None or self.biased or self.values_from_keys
+                                or self.query_temperature is not None):
+            raise ValueError("attention: a norm over the projection needs qk_norm_eps and does not combine with biases, "
+                             "values from keys or a query temperature")
         self.bias = {"q": None, "k": None, "v": None}
         if self.num_heads % self.num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
@@ -159,7 +175,7 @@ class Attention(Mixer):
         if self.neighbours and self.position is not None and \
                 int(getattr(self.position, "rotary_dim", 0)) > self.head_dim:
             raise ValueError("attention: the rotation covers more values than a head has")
-        self.w_qkv = self.w_o = self.q_gain = self.k_gain = None
+        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.sinks = None
 
     def cache_spec(self):
         window = self.spec.params.get("cache_window") or self.window or self.chunk
@@ -209,9 +225,12 @@ class Attention(Mixer):
             n = self.num_heads if which == "q" else self.num_kv_heads
             self.bias[which] = self._by_head(tensors[w[which + "_bias"]].to(f32), n, which != "v").contiguous()
         if self.qk_norm_eps is not None:
-            self.q_gain = self._by_head(tensors[w["q_norm"]].to(f32), 1, True).contiguous()
+            heads = (self.num_heads, self.num_kv_heads) if self.whole_norm else (1, 1)
+            self.q_gain = self._by_head(tensors[w["q_norm"]].to(f32), heads[0], True).contiguous()
             if self.kv_projection:
-                self.k_gain = self._by_head(tensors[w["k_norm"]].to(f32), 1, True).contiguous()
+                self.k_gain = self._by_head(tensors[w["k_norm"]].to(f32), heads[1], True).contiguous()
+        if self.has_sinks:
+            self.sinks = tensors[w["sink"]].to(f32).contiguous()
         if self.output_biased:
             self.output_bias = tensors[w["o_bias"]].to(f32).contiguous()
 
@@ -243,7 +262,9 @@ class Attention(Mixer):
         rows = linear(x, self.w_qkv, ctx, "qkv", n_rows=t)
         k_col = nh * big
         gate_col = k_col + (2 * nkv * big if self.kv_projection else 0)
-        if self.qk_norm_eps is not None or self.biased:
+        if self.whole_norm:
+            self._whole_norm_kv(rows, ctx, entry, writes_cache and self.kv_projection)
+        elif self.qk_norm_eps is not None or self.biased:
             kernels.qk_prepare_padded_kv(
                 rows, t, self.q_gain, self.k_gain, pos.cos if pos else _no_table(self.device),
                 pos.sin if pos else _no_table(self.device), pos.rotary_dim if pos else 0, ctx.positions,
@@ -261,7 +282,7 @@ class Attention(Mixer):
         out = ctx.workspace.get("attn_out", (t, nh * big), self.dtype)
         visible = self._visible(ctx)
         gate = rows[:, gate_col:] if self.head_gate else None
-        mask = {"chunk": self.chunk, "softcap": self.softcap}
+        mask = {"chunk": self.chunk, "softcap": self.softcap, "sinks": self.sinks}
         if not ctx.is_decode and kernels.attention_prefill_supported(self.dtype, big, nh, nkv):
             kernels.attention_prefill_bf16(out, rows, t, ctx.positions, ctx.token_slot, ctx.cu_seqlens, ctx.n_seqs,
                                            entry.k_pages, entry.v_pages, entry.block_table, nh, nkv, big, self.scale,
@@ -295,6 +316,14 @@ class Attention(Mixer):
                                   acc, ml, keep_first=self.keep_first, gate=gate, **mask)
         return self._project(out, ctx, None, leave_bias)
 
+    def _whole_norm_kv(self, rows, ctx, entry, write_kv):
+        pos = self.position
+        kernels.qk_whole_norm_kv(
+            rows, ctx.n_tokens, self.q_gain, self.k_gain, pos.cos if pos else _no_table(self.device),
+            pos.sin if pos else _no_table(self.device), pos.rotary_dim if pos else 0, ctx.positions, ctx.token_slot,
+            entry.k_pages, entry.v_pages, entry.block_table, self.num_heads, self.num_kv_heads, self.padded_dim,
+            self.qk_norm_eps, norm_dim=self.head_dim, write_kv=write_kv)
+
     def load(self, tensors):
         if self.general:
             return self._load_general(tensors)
@@ -310,7 +339,7 @@ class Attention(Mixer):
 
     def bytes_read_per_step(self, n_tokens):
         return sum(t.numel() * t.element_size() for t in (self.w_qkv, self.w_o, self.q_gain, self.k_gain,
-                                                          self.output_bias, *self.bias.values()) if t is not None)
+                                                          self.sinks, self.output_bias, *self.bias.values()) if t is not None)
 
     # ------------------------------------------------------------------
     takes_deferred_norm = True
@@ -384,7 +413,9 @@ class Attention(Mixer):
                    pos.rotary_dim if pos else 0, ctx.positions, ctx.token_slot, entry.k_pages,
                    entry.v_pages, entry.block_table, self.num_heads, self.num_kv_heads, self.head_dim,
                    self.qk_norm_eps if self.qk_norm_eps is not None else 0.0)
-        if self._plain:
+        if self.whole_norm:
+            self._whole_norm_kv(qkv, ctx, entry, writes_cache)
+        elif self._plain:
             kernels.qk_norm_rope_kv(*prepare, write_kv=writes_cache)
         else:
             kernels.qk_prepare_kv(*prepare, write_kv=writes_cache, q_bias=self.bias["q"],
@@ -398,8 +429,8 @@ class Attention(Mixer):
     @property
     def _plain(self):
         """None of the optional parameters that change what happens between the projection and
-        the cache is on (the sink only changes the softmax)."""
-        return not self.biased and not self.values_from_keys and self.query_temperature is None
+        the cache is on (sinks only change the softmax)."""
+        return not self.biased and not self.values_from_keys and self.query_temperature is None and not self.whole_norm
 
     def _fuses_rope(self, x, ctx):
         xin = x.scaled if isinstance(x, DeferredNorm) else x
@@ -411,7 +442,7 @@ class Attention(Mixer):
     def product_image(self):
         """``"extended"`` when this layer's q/k/v product of few rows runs the extended epilogue."""
         pos = self.position
-        if ((not self._plain or pos is None) and self.dtype == torch.bfloat16
+        if ((not self._plain or pos is None) and not self.whole_norm and self.dtype == torch.bfloat16
                 and self.head_dim == kernels.QKV_ROPE_HEAD_DIM
                 and (pos is None or getattr(pos, "rotary_dim", 0) == self.head_dim)):
             return "extended"
@@ -434,7 +465,7 @@ class Attention(Mixer):
     def _attend(self, out, qkv, ctx, entry):
         t = ctx.n_tokens
         visible = self._visible(ctx)
-        mask = {"chunk": self.chunk, "softcap": self.softcap}
+        mask = {"chunk": self.chunk, "softcap": self.softcap, "sinks": self.sinks}
         fast_decode = ctx.is_decode and kernels.attention_decode_supported(self.dtype, self.head_dim)
         if not ctx.is_decode and kernels.attention_prefill_supported(
                 self.dtype, self.head_dim, self.num_heads, self.num_kv_heads):

@@ -16,6 +16,11 @@ times ``scale``, not divided by their sum.  With ``weigh="input"`` the weight mu
 its output: out = sum over the chosen experts of W_down,e act(W_up,e (weight h)); the product is linear, so the
 weight joins it in the 32-bit sums.  ``shared``, a feed-forward PartSpec, runs for every token and is added.
 
+With ``weights="softmax"`` the weights are the chosen scores of the softmax over all experts, times ``scale`` and not
+divided by their sum; with ``corrected`` a learned number per expert (tensor ``correction`` [E + identity], any sign)
+joins the scores for the choice, not for the weights.  ``identity`` more experts without tensors stand behind the others
+in the router: such an expert's output is the input itself.
+
 Experts have no biases; ``activation`` is ``"relu2"`` (the square of relu), ``"silu"``,
 ``"gelu_tanh"``, ``"none"`` or, for gated experts, ``"clamped"`` with a ``limit`` (``parts/mlp.py``).  The choice is made and used on the device: a kernel sorts the (token,
 choice) pairs by expert and cuts every expert's stretch into row tiles, and the two expert products
@@ -23,8 +28,8 @@ walk those tiles, so nothing here waits for the device and the step can be captu
 
 Parameters: ``hidden_size``, ``intermediate_size`` (of one expert), ``experts``, ``top``, ``groups``
 (default 1), ``keep`` (default: all groups), ``scale``, ``activation``, ``gated`` (default False), ``weights``
-(``"scores_of_chosen"``, the default, ``"softmax_of_chosen"`` or ``"sigmoid"``), ``weigh`` (``"output"``, the default, or
-``"input"``), ``limit``, ``shared``.  Tensors: ``router`` [E, hidden]
+(``"scores_of_chosen"``, the default, ``"softmax_of_chosen"``, ``"sigmoid"`` or ``"softmax"``), ``weigh`` (``"output"``, the default, or
+``"input"``), ``limit``, ``shared``, ``corrected``, ``identity`` (default 0).  Tensors: ``router`` [E + identity, hidden]
 and per expert ``up_<e>`` [I, hidden], ``down_<e>`` [hidden, I].
 """
 
@@ -45,7 +50,9 @@ class RoutedExperts(FeedForward):
     def tensors(cls, spec):
         p, w = spec.params, spec.weights
         h, i, n = p["hidden_size"], p["intermediate_size"], p["experts"]
-        out = [TensorSpec(w["router"], (n, h))]
+        out = [TensorSpec(w["router"], (n + int(p.get("identity") or 0), h))]
+        if p.get("corrected"):
+            out.append(TensorSpec(w["correction"], (n + int(p.get("identity") or 0),), "around_zero"))
         for e in range(n):
             if p.get("gated"):
                 out.append(TensorSpec(w[f"gate_{e}"], (i, h)))
@@ -67,6 +74,9 @@ class RoutedExperts(FeedForward):
         self.weights = spec.params.get("weights", "scores_of_chosen")
         self.weigh_input = spec.params.get("weigh", "output") == "input"
         self.limit = float(spec.params.get("limit") or 0.0)
+        self.identity = int(spec.params.get("identity") or 0)
+        self.corrected = bool(spec.params.get("corrected"))
+        self.routed = self.experts + self.identity           # what the router chooses among
         shared = spec.params.get("shared")
         self.shared = None if shared is None else lookup_part("feed_forward", shared.kind)(shared, dtype, device)
         if spec.params.get("weigh", "output") not in ("output", "input"):
@@ -77,10 +87,15 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"routed_experts has no weights {self.weights!r}")
         if self.activation not in kernels.EXPERT_ACTIVATIONS:
             raise ValueError(f"routed_experts has no activation {self.activation!r}")
-        if self.experts % self.groups or not 1 <= self.keep <= self.groups:
+        if self.routed % self.groups or not 1 <= self.keep <= self.groups:
             raise ValueError("routed_experts: groups must divide experts, 1 <= keep <= groups")
-        if not 1 <= self.top <= self.keep * (self.experts // self.groups):
+        if not 1 <= self.top <= self.keep * (self.routed // self.groups):
             raise ValueError("routed_experts: top exceeds the experts of the kept groups")
+        if self.corrected and self.weights != "softmax":
+            raise ValueError("routed_experts: a correction of the choice goes with the weights 'softmax'")
+        if self.identity < 0 or (self.identity and self.weigh_input):
+            raise ValueError("routed_experts: identity experts are counted from 0 and are weighed on their output")
+        self.correction = None
         self.w_router = self.w_up = self.w_down = None
 
     def load(self, tensors):
@@ -88,6 +103,8 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             self.shared.load(tensors)
         self.w_router = tensors[w["router"]].to(self.dtype).contiguous()
+        if self.corrected:
+            self.correction = tensors[w["correction"]].to(torch.float32).contiguous()
         ups = [tensors[w[f"up_{e}"]] for e in range(self.experts)]
         if self.gated:               # rows gate_0, up_0, gate_1, up_1, ... of every expert
             ups = [torch.stack([tensors[w[f"gate_{e}"]], up], 1).reshape(2 * self.inter, self.hidden)
@@ -109,7 +126,7 @@ class RoutedExperts(FeedForward):
         chosen = ws.get("moe_chosen", (t, top), torch.int32)
         weight = ws.get("moe_weight", (t, top), torch.float32)
         kernels.moe_route(chosen, weight, logits, t, self.groups, self.keep, top, self.scale,
-                          weights=self.weights)
+                          weights=self.weights, correction=self.correction)
         sorted_pair = ws.get("moe_sorted", (pairs,), torch.int32)
         tiles = ws.get("moe_tiles", (kernels.moe_max_tiles(pairs, self.experts), 3), torch.int32)
         n_tiles = ws.get("moe_n_tiles", (1,), torch.int32)
@@ -125,5 +142,6 @@ class RoutedExperts(FeedForward):
             self.shared.product_image = self.product_image
             add = self.shared.forward(x, ctx)
         out = ws.get("moe_out", (t, self.hidden), self.dtype)
-        kernels.moe_combine(out, pair_out, t, top, add=add)
+        kernels.moe_combine(out, pair_out, t, top, add=add,
+                            identity=(chosen, weight, x, self.experts) if self.identity else None)
         return out

@@ -1,5 +1,5 @@
 """Two recurrent mixers with a decay per head and token, over one scan kernel, one over the same kernel whose
-decays are constants of the heads (``fixed_decay_memory``), and one with a decay per channel and no matrix state
+decays are constants of the heads (``fixed_decay_memory``; ``retention`` with rotated keys), and one with a decay per channel and no matrix state
 (``gated_linear_recurrence``; both described at their classes).
 
 Both keep a matrix S [key size, value size] per head and sequence in 32-bit and update it token by token,
@@ -45,7 +45,7 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import linear
-from ..registry import register_part
+from ..registry import lookup_part, register_part
 from .base import Mixer
 from .spec import CacheSpec, TensorSpec
 
@@ -241,6 +241,76 @@ class FixedDecayMemory(Mixer):
                            ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache, n_tokens=t)
         y = ws.get("attn_out", (t, nh * e), self.dtype)
         kernels.norm_gate_out(y, o, proj, width, self.norm_w, self.eps, ctx.positions, t)
+        return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
+
+
+@register_part("mixer", "retention")
+class Retention(Mixer):
+    """Linear attention with fixed decays and rotated queries and keys (the retention of RetNet).  H heads, key size d,
+    value size e:
+
+        q = rot(W_q h), k = rot(W_k h), v = W_v h
+        S_t = decay_head S_(t-1) + d^-1/2 k_t v_t^T;   o_t = S_t^T q_t      (S from zero, 32-bit; no softmax, no denominator)
+        y = o / rms(o) per head (no weight) * silu(W_g h);   out = W_o y
+
+    The factor d^-1/2 is the scan's b; projections, rotation, S and the norm are 32-bit, y is rounded once to the
+    activation type.  Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``v_dim``, ``decay`` (H numbers),
+    ``eps``, ``position`` (a rotary PartSpec, or None).  Tensors: ``q``, ``k`` [H d, hidden], ``v``, ``g`` [H e, hidden],
+    ``o`` [hidden, H e]."""
+
+    @classmethod
+    def tensors(cls, spec):
+        p, w = spec.params, spec.weights
+        hid, nh, d, e = p["hidden_size"], p["num_heads"], p["head_dim"], p["v_dim"]
+        return [TensorSpec(w["q"], (nh * d, hid)), TensorSpec(w["k"], (nh * d, hid)), TensorSpec(w["v"], (nh * e, hid)),
+                TensorSpec(w["g"], (nh * e, hid)), TensorSpec(w["o"], (hid, nh * e))]
+
+    def __init__(self, spec, dtype, device):
+        super().__init__(spec, dtype, device)
+        g = lambda n: int(self.param(n))
+        self.hidden, self.num_heads, self.head_dim, self.v_dim = g("hidden_size"), g("num_heads"), g("head_dim"), g("v_dim")
+        self.eps = float(self.param("eps"))
+        self.decay = [float(x) for x in self.param("decay")]
+        if len(self.decay) != self.num_heads:
+            raise ValueError("retention: one decay per head")
+        pos = spec.params.get("position")
+        self.position = lookup_part("position", pos.kind)(pos, dtype, device) if pos else None
+        if self.position is not None and self.position.rotary_dim > self.head_dim:
+            raise ValueError("retention: the rotation covers more values than a head has")
+        self.rows = kernels.decay_scan_rows(self.head_dim)
+        self.s_values = self.num_heads * self.v_dim * self.rows
+        self.w_in = self.w_o = self.a = self.b = None
+
+    def cache_spec(self):
+        return CacheSpec("state", shape=(-(-self.s_values // 4) * 4,))
+
+    def prepare(self, max_positions):
+        if self.position is not None:
+            self.position.prepare(max_positions)
+
+    def load(self, tensors):
+        w, f32 = self.spec.weights, torch.float32
+        rows = [tensors[w[n]] for n in ("q", "k", "v", "g")]
+        self.w_in = _padded_rows(rows, self.hidden).to(self.dtype).contiguous()
+        self.w_o = tensors[w["o"]].to(self.dtype).contiguous()
+        self.a = torch.tensor(self.decay, dtype=f32, device=self.device)
+        self.b = torch.full_like(self.a, self.head_dim ** -0.5)
+
+    def bytes_read_per_step(self, n_tokens):
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o))
+
+    def forward(self, x, ctx, entry, writes_cache=True):
+        t, ws, f32 = ctx.n_tokens, ctx.workspace, torch.float32
+        nh, d, e, pos = self.num_heads, self.head_dim, self.v_dim, self.position
+        proj = linear(x, self.w_in, ctx, "retention_in", n_rows=t, out_dtype=f32, wide_f32="library")
+        if pos is not None:                                  # query and key heads stand side by side
+            kernels.rotate_heads(proj, 0, 2 * nh, d, pos.rotary_dim, pos.cos, pos.sin, ctx.positions, t)
+        o = ws.get("scan_o", (t, nh * e), f32)
+        kernels.decay_scan(o, proj, proj[:, nh * d:], proj[:, 2 * nh * d:], self.a, self.b, entry.state, ctx.cu_seqlens,
+                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache, n_tokens=t)
+        y = ws.get("attn_out", (t, nh * e), self.dtype)
+        kernels.head_norm_gate_out(y, o, proj, nh * (2 * d + e), None, self.eps, ctx.positions, t, nh, e,
+                                   gate_activation="silu")
         return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
 
 

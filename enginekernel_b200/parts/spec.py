@@ -113,6 +113,8 @@ class ModelSpec:
     position_table: Optional[TensorSpec] = None
     #: logits = logit_multiplier * (final norm . lm_head^T)
     logit_multiplier: float = 1.0
+    #: then logits = cap * tanh(logits / cap) (None: no cap)
+    logit_softcap: Optional[float] = None
     #: tensor names a checkpoint may hold although the model does not read them
     ignorable: Tuple[str, ...] = ()
     #: a hashed table of token pairs added to the embedding (None: the model has none)
@@ -134,6 +136,8 @@ class ModelSpec:
                                                                                      self.hidden_size):
             raise ValueError(f"the position table must be [{self.max_positions}, {self.hidden_size}], "
                              f"not {tuple(self.position_table.shape)}")
+        if self.logit_softcap is not None and not self.logit_softcap > 0:
+            raise ValueError("the soft cap of the logits must be positive")
         if self.input_mix is not None and tuple(self.input_mix.shape) != (self.hidden_size, 2 * self.hidden_size):
             raise ValueError(f"input_mix must be [{self.hidden_size}, {2 * self.hidden_size}], "
                              f"not {tuple(self.input_mix.shape)}")
