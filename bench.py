@@ -7,6 +7,7 @@
     python bench.py --design bolelix [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
     python bench.py --design musavik [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
     python bench.py --design kamosun [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
+    python bench.py --design gesuvik [--sizes 1b,2b] [--layers L] [--batch B] [--skip-kernels]
 
 The shapes and workloads are the ones BASELINE.json names (its configs[2], [3], [4]):
 
@@ -39,6 +40,9 @@ Bolelix decoder of the same width and layer count.
 ``--design kamosun`` measures the Kamosun decoder (a pair of full attention and fixed-decay memory, then three layers of
 chunked attention, one of which reads another's keys, all with gated results, averages over the depth and routed
 experts beside a shared one) next to the Bolelix decoder of the same width, layer count and experts.
+``--design gesuvik`` measures the Gesuvik decoder (retention, windowed latent attention, retention and windowed
+attention in turn, every one with routed experts, some of them the identity, beside a shared one) next to the Kamosun
+decoder of the same width, layer count, heads and experts.
 One line of JSON is printed.  The inputs of a step (gigabytes of weights) are larger than
 the L2.
 
@@ -524,10 +528,48 @@ def kamosun_configs(size: dict, layers: int, context: int):
     return kamosun, bolelix_configs(BOLELIX_SIZES[size["beside"]], layers, context)[0]
 
 
+# Gesuvik at sizes that resemble real layers, beside the Kamosun decoder - the closest design here: it too mixes
+# attention over a part of the context with linear attention over the decay scan, and has clamped gated experts beside a
+# shared one - at the same width, layer count, head sizes and experts.  Layers in turn: retention, latent attention,
+# retention, attention.
+GESUVIK_SIZES = {
+    "1b": dict(width=2048, vocab=128256, retention=dict(heads=16, dim=128, vdim=128),
+               latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=192, window=1024),
+               attention=dict(heads=16, kv_heads=8, dim=128, vdim=128, rot=128, window=1024),
+               moe=dict(experts=32, identity=8, ff=1024, top=4, shared=1024), beside="1b"),
+    "2b": dict(width=2560, vocab=151936, retention=dict(heads=10, dim=256, vdim=256),
+               latent=dict(heads=20, dim=128, rot_dim=64, vdim=192, kv_rank=160, window=512),
+               attention=dict(heads=20, kv_heads=10, dim=128, vdim=128, rot=64, window=512),
+               moe=dict(experts=16, identity=4, ff=1536, top=2, shared=2048), beside="2b"),
+}
+
+
+def gesuvik_configs(size: dict, layers: int, context: int):
+    """(Gesuvik configuration, Kamosun configuration) of one size."""
+    from enginekernel_b200.config.gesuvik import GesuvikConfig
+    at, la, re_, m = size["attention"], size["latent"], size["retention"], size["moe"]
+    moe = {"kind": "moe", "expert": {"ff": m["ff"], "limit": 7.0}, "shared": {"ff": m["shared"], "limit": 7.0},
+           "router": {"experts": m["experts"], "identity": m["identity"], "top": m["top"]}}
+    attention = {"dim": at["dim"], "vdim": at["vdim"], "heads": at["heads"], "kv_heads": at["kv_heads"],
+                 "scale": at["dim"] ** -0.5, "mask": {"size": at["window"]},
+                 "rot": {"base": 1000000.0, "dims": at["rot"],
+                         "scaling": {"factor": 4.0, "fast": 32.0, "original": 8192, "slow": 1.0}}}
+    latent = {"heads": la["heads"], "dim": la["dim"], "rot_dim": la["rot_dim"], "vdim": la["vdim"],
+              "kv_rank": la["kv_rank"], "scale": (la["dim"] + la["rot_dim"]) ** -0.5, "mask": {"size": la["window"]},
+              "rot": {"base": 1000000.0, "dims": la["rot_dim"]}}
+    retention = dict(re_, decay=[1.0 - 2.0 ** (-5.0 - 6.0 * h / re_["heads"]) for h in range(re_["heads"])],
+                     rot={"base": 10000.0, "dims": re_["dim"]})
+    turn = [("retention", retention), ("latent_attention", latent), ("retention", retention), ("attention", attention)]
+    made = [{"type": turn[i % 4][0], "mixer": turn[i % 4][1], "mlp": moe} for i in range(layers)]
+    gesuvik = GesuvikConfig.from_dict({"architecture": "Gesuvik", "vocab": size["vocab"], "width": size["width"],
+                                       "norm": {"eps": 1e-6}, "logit_scale": 0.5, "logit_softcap": 30.0, "layers": made})
+    return gesuvik, kamosun_configs(KAMOSUN_SIZES[size["beside"]], layers, context)[0]
+
+
 #: design -> (sizes, configurations of one size, the design it is measured beside)
 DESIGNS = {"lopazen": (DESIGN_SIZES, design_configs, "qwen3"), "susalorn": (SUSALORN_SIZES, susalorn_configs, "qwen3"),
            "bolelix": (BOLELIX_SIZES, bolelix_configs, "susalorn"), "musavik": (MUSAVIK_SIZES, musavik_configs, "bolelix"),
-           "kamosun": (KAMOSUN_SIZES, kamosun_configs, "bolelix")}
+           "kamosun": (KAMOSUN_SIZES, kamosun_configs, "bolelix"), "gesuvik": (GESUVIK_SIZES, gesuvik_configs, "kamosun")}
 
 
 def measure_design(cfg, vocab, batch, prompt_len, context, steps, warmup, pk, with_kernels):
@@ -653,9 +695,9 @@ def main(argv=None) -> int:
     ap.add_argument("--skip-kernels", action="store_true", help="leave out the per-kernel tables")
     ap.add_argument("--prefill-seqs", type=int, default=1,
                     help="sequences of 2,048 tokens in the prompt step of the per-kernel table")
-    ap.add_argument("--design", default="", choices=["", "lopazen", "susalorn", "bolelix", "musavik", "kamosun"],
+    ap.add_argument("--design", default="", choices=["", "lopazen", "susalorn", "bolelix", "musavik", "kamosun", "gesuvik"],
                     help="instead of the default workload: this design beside the Qwen3 decoder (bolelix: beside "
-                         "the Susalorn decoder; musavik, kamosun: beside the Bolelix decoder) at equal layer sizes (prompt "
+                         "the Susalorn decoder; musavik, kamosun: beside the Bolelix decoder; gesuvik: beside the Kamosun decoder) at equal layer sizes (prompt "
                          "step, decode step, per-kernel tables)")
     ap.add_argument("--sizes", default="", help="with --design: comma-separated names of DESIGN_SIZES")
     args = ap.parse_args(argv)
