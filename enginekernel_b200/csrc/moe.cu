@@ -41,10 +41,10 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 
 constexpr int kRouteWarps = 4;
 
-// logits [T, E] 32-bit -> sel_expert [T, top] int32, sel_weight [T, top] 32-bit.
+// logits [T, >= E] 32-bit (rows row_stride apart) -> sel_expert [T, top] int32, sel_weight [T, top] 32-bit.
 __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
-                 const float* __restrict__ logits, int n_tokens, int E, int n_groups, int keep, int top,
+                 const float* __restrict__ logits, int row_stride, int n_tokens, int E, int n_groups, int keep, int top,
                  float scale, int mode, const float* __restrict__ correction) {
   // mode 0: softmax scores, divided by the chosen ones' sum; 1: softmax over the chosen; 2: sigmoids as they are;
   // 3: softmax scores as they are, chosen by score + correction
@@ -58,7 +58,7 @@ moe_route_kernel(int* __restrict__ sel_expert, float* __restrict__ sel_weight,
   float* s = route_s + (size_t)warp * (2 * E + n_groups);
   float* cand = s + E;
   float* gs = cand + E;
-  const float* z = logits + (size_t)t * E;
+  const float* z = logits + (size_t)t * row_stride;
   float m = -INFINITY;
   for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
   m = warp_max(m);
@@ -435,20 +435,19 @@ moe_combine_kernel(T* __restrict__ out, const float* __restrict__ pair_out, int 
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
-  if (vec) {
+  if (vec) {                                     // (top <= 32: which choices are the input itself, one bit each)
+    unsigned own = 0;
+    if (chosen)
+      for (int k = 0; k < top; ++k) own |= (chosen[t * top + k] >= E ? 1u : 0u) << k;
     for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      const float4 xv = chosen ? Vec4<T>::load(x + t * width + i) : a;
+      const float4 xv = own ? Vec4<T>::load(x + t * width + i) : a;
 #pragma unroll 4
       for (int k = 0; k < top; ++k) {
-        float w = 1.f;
-        float4 v;
-        if (chosen && chosen[t * top + k] >= E) {
-          w = weight[t * top + k];
-          v = xv;
-        } else {
-          v = *reinterpret_cast<const float4*>(pair_out + (t * top + k) * width + i);
-        }
+        const bool mine = own >> k & 1u;
+        float4 v = xv;
+        if (!mine) v = *reinterpret_cast<const float4*>(pair_out + (t * top + k) * width + i);
+        const float w = mine ? weight[t * top + k] : 1.f;
         a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
       }
       if (add) {
@@ -473,12 +472,12 @@ moe_combine_kernel(T* __restrict__ out, const float* __restrict__ pair_out, int 
 
 EK_EXPORT int ek_moe_tile_rows() { return ek::kTileRows; }
 
-EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logits, int n_tokens, int E,
+EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logits, int row_stride, int n_tokens, int E,
                            int n_groups, int keep, int top, float scale, int mode,
                            const float* correction, cudaStream_t stream) {
   using namespace ek;
   if (n_tokens <= 0) return 0;
-  if (E <= 0 || top <= 0 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
+  if (E <= 0 || row_stride < E || top <= 0 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
       top > keep * (E / n_groups) || mode < 0 || mode > 3 || (mode >= 2 && keep < n_groups) ||
       (correction && mode != 3))
     return EK_ERR_ARG;
@@ -489,7 +488,7 @@ EK_EXPORT int ek_moe_route(int* sel_expert, float* sel_weight, const float* logi
     if (e != cudaSuccess) return (int)e;
   }
   moe_route_kernel<<<(n_tokens + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, stream>>>(
-      sel_expert, sel_weight, logits, n_tokens, E, n_groups, keep, top, scale, mode, correction);
+      sel_expert, sel_weight, logits, row_stride, n_tokens, E, n_groups, keep, top, scale, mode, correction);
   EK_RETURN_LAUNCH_STATUS();
 }
 
@@ -570,7 +569,7 @@ EK_EXPORT int ek_moe_expert_down_tc(float* out, const void* a, const void* w, co
     if (n_tokens <= 0) return 0;                                                                      \
     if (width <= 0 || top <= 0 || (chosen && (!weight || !x))) return EK_ERR_ARG;                     \
     const uintptr_t rows = (uintptr_t)out | (uintptr_t)add | (uintptr_t)x;                            \
-    const int vec = width % 4 == 0 && ((uintptr_t)pair_out & 15) == 0 && (rows & (4 * sizeof(T) - 1)) == 0; \
+    const int vec = width % 4 == 0 && top <= 32 && ((uintptr_t)pair_out & 15) == 0 && (rows & (4 * sizeof(T) - 1)) == 0; \
     ek::moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>((T*)out, pair_out, top, width, (const T*)add, \
                                                             chosen, weight, (const T*)x, E, vec);     \
     EK_RETURN_LAUNCH_STATUS();                                                                        \

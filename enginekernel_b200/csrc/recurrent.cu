@@ -452,52 +452,117 @@ xgate_scan_kernel(float* __restrict__ a, float* __restrict__ b, float* __restric
   if (write_state && threadIdx.x == 0) *m_state = m_in;
 }
 
-constexpr int kScanCols = 16;        // columns of S a block takes
+constexpr int kScanCols = 16;        // columns of S a block takes (twice as many with two a lane)
 constexpr int kScanLanes = 8;        // lanes that share a column
 constexpr int kScanThreads = kScanCols * kScanLanes;
 constexpr int kScanFloats = 2048;    // values of keys (and of queries) fetched into shared memory at a time
+
+// Long prompts of few sequences leave most of the machine empty when every sequence is walked by one block a head and
+// tile, so they are cut into segments of `seg_len` tokens that are walked side by side: a first launch (MODE 1) runs
+// every segment but a sequence's last from S = 0 (the first one from the sequence's state) and keeps what it ends with
+// and the product of its decays; the second (MODE 2) starts every segment from what the ones before it leave together,
+//     S_in(0) = state,  S_in(1) = X_1,  S_in(p + 1) = prod_p S_in(p) + X_(p+1),
+// which is the recurrence itself with its sums taken in another order.  MODE 0 is the whole walk in one launch.
+// `carry` [sequence][segment][heads][C][DK]: slot 0 a copy of the state (the second launch may replace it while other
+// blocks still need it), slot p + 1 the end of segment p; `prods` [sequence][segment][heads].
+struct ScanSegments {
+  float* carry;
+  float* prods;
+  int count;                 // segments of the longest sequence (grid.x = sequences * count)
+  int len;
+};
 
 // grid (sequences, heads, column tiles).  RPL rows of a column a lane: lane l holds rows 32 g + 4 l + c
 // (g < RPL / 4, c < 4), so that the 8 lanes of a column read 128 neighbouring bytes of a key at a time.
 // S of a slot: state[((h * C + j) * DK + i], DK = 8 RPL rows (keys padded with zeros), C = dv + ones_col columns.
 // `ab_stride`: values of a (and b) from token to token - the heads, or 0 where they are the same for every token.
+// CPL columns a lane (j and j + 16): with two, a key fetched from shared memory - what bounds a long walk - serves two
+// columns; single tokens take one, for the shorter walk through S.
 // Column dv (with ones_col) has v = 1: it carries n_t = a n + b k and gives n.q.
 // Tokens come 2048 / DK at a time: while one portion is worked through from shared memory, the next one's
 // keys, queries, values and gates are already on their way into registers.
-template <int RPL>
+template <int RPL, int MODE, int CPL>
 __global__ void __launch_bounds__(kScanThreads)
 decay_scan_kernel(float* __restrict__ out, int out_stride, const float* __restrict__ q, int q_stride,
                   const float* __restrict__ k, int k_stride, const float* __restrict__ v, int v_stride,
                   const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ state,
                   size_t slot_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ positions,
                   const int* __restrict__ token_slot, int heads, int kv_heads, int dk, int dv, int ones_col,
-                  int write_state, int ab_stride) {
-  constexpr int DK = 8 * RPL, G4 = RPL / 4, DK4 = DK / 4;
+                  int write_state, int ab_stride, ScanSegments seg) {
+  constexpr int DK = 8 * RPL, G4 = RPL / 4, DK4 = DK / 4, COLS = kScanCols * CPL;
   constexpr int CH = kScanFloats / DK;                       // tokens a portion: 64, 32, 16 or 8
   constexpr int NV4 = kScanFloats / 4 / kScanThreads;        // float4 of keys (of queries) a thread fetches
-  constexpr int NV = CH * kScanCols / kScanThreads;          // values a thread fetches
-  static_assert(CH <= kScanThreads && CH * kScanCols % kScanThreads == 0, "portion sizes");
+  constexpr int NV = CH * COLS / kScanThreads;               // values a thread fetches
+  static_assert(CH <= kScanThreads && CH * COLS % kScanThreads == 0, "portion sizes");
   __shared__ __align__(16) float k_s[CH][DK];
   __shared__ __align__(16) float q_s[CH][DK];
-  __shared__ float v_s[CH][kScanCols];
+  __shared__ float v_s[CH][COLS];
   __shared__ float a_s[CH], b_s[CH];
   pdl_launch_dependents();
   pdl_wait();
-  const int seq = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kScanCols;
-  const int start = cu_seqlens[seq], n = cu_seqlens[seq + 1] - start;
+  const int seq = MODE == 0 ? blockIdx.x : blockIdx.x / seg.count, part = MODE == 0 ? 0 : blockIdx.x % seg.count;
+  const int h = blockIdx.y, col0 = blockIdx.z * COLS;
+  int start = cu_seqlens[seq], n = cu_seqlens[seq + 1] - start;
   if (n <= 0 || positions[start] < 0) return;
+  const int slot = token_slot[start];
+  bool alone = MODE == 0;                        // one block a head and tile walks the whole sequence
+  if (MODE != 0) {                               // this block's segment
+    const int parts = (n + seg.len - 1) / seg.len;
+    if (part >= (MODE == 1 ? parts - 1 : parts)) return;
+    alone = parts == 1;
+    if (part < parts - 1) write_state = 0;       // (the last segment's end is the sequence's new state)
+    start += part * seg.len;
+    n = min(seg.len, n - part * seg.len);
+  }
   const int tid = threadIdx.x, col = tid / kScanLanes, lane = tid % kScanLanes;
-  const int C = dv + ones_col, j = col0 + col;
-  const bool live = j < C;
+  const int C = dv + ones_col;
+  int j[CPL];
+  bool live[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    j[c] = col0 + col + c * kScanCols;
+    live[c] = j[c] < C;
+  }
   const int kv = h / (heads / kv_heads);
   // whole float4 loads need rows and head offsets on 16-byte boundaries
   const bool vec = dk % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 &&
                    (((uintptr_t)q | (uintptr_t)k) & 15) == 0;
-  float* sp = state + (size_t)token_slot[start] * slot_stride + ((size_t)h * C + (live ? j : 0)) * DK;
-  float4 S[G4];
+  float* sp = state + (size_t)slot * slot_stride;
+  auto carry_at = [&](int slot_of) { return seg.carry + ((size_t)seq * seg.count + slot_of) * heads * C * DK; };
+  auto place = [&](int c, int g) { return ((size_t)h * C + j[c]) * DK + 32 * g + 4 * lane; };     // of S within a slot
+  auto load = [&](const float* from, int c, int g) { return *reinterpret_cast<const float4*>(from + place(c, g)); };
+  auto store = [&](float* to, int c, int g, float4 v) { *reinterpret_cast<float4*>(to + place(c, g)) = v; };
+  float4 S[CPL][G4];
+  {
+    const float* from = MODE == 2 && !alone ? carry_at(min(part, 1)) : sp;
 #pragma unroll
-  for (int g = 0; g < G4; ++g)
-    S[g] = live ? *reinterpret_cast<const float4*>(sp + 32 * g + 4 * lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c = 0; c < CPL; ++c)
+#pragma unroll
+      for (int g = 0; g < G4; ++g)
+        S[c][g] = !live[c] || (MODE == 1 && part > 0) ? make_float4(0.f, 0.f, 0.f, 0.f) : load(from, c, g);
+  }
+  if (MODE == 1 && part == 0) {
+#pragma unroll
+    for (int c = 0; c < CPL; ++c)
+#pragma unroll
+      for (int g = 0; g < G4; ++g)
+        if (live[c]) store(carry_at(0), c, g, S[c][g]);
+  }
+  if (MODE == 2) {
+    for (int i = 2; i <= part; ++i) {            // X_1, then one segment after another
+      const float f = seg.prods[((size_t)seq * seg.count + i - 1) * heads + h];
+      const float* x = carry_at(i);
+#pragma unroll
+      for (int c = 0; c < CPL; ++c)
+#pragma unroll
+        for (int g = 0; g < G4; ++g) {
+          if (!live[c]) continue;
+          const float4 e = load(x, c, g), o = S[c][g];
+          S[c][g] = make_float4(fmaf(f, o.x, e.x), fmaf(f, o.y, e.y), fmaf(f, o.z, e.z), fmaf(f, o.w, e.w));
+        }
+    }
+  }
+  float prod = 1.f;                              // MODE 1: the segment's decays together
 
   float4 k_r[NV4], q_r[NV4];
   float v_r[NV], a_r = 1.f, b_r = 0.f;
@@ -522,12 +587,12 @@ decay_scan_kernel(float* __restrict__ out, int out_stride, const float* __restri
       k_r[m] = q_r[m] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (tt < nc) {
         row4(k_r[m], k, (size_t)start + c0 + tt, k_stride, i);
-        row4(q_r[m], q, (size_t)start + c0 + tt, q_stride, i);
+        if (MODE != 1) row4(q_r[m], q, (size_t)start + c0 + tt, q_stride, i);
       }
     }
 #pragma unroll
     for (int m = 0; m < NV; ++m) {
-      const int f = tid + m * kScanThreads, tt = f / kScanCols, jj = col0 + f % kScanCols;
+      const int f = tid + m * kScanThreads, tt = f / COLS, jj = col0 + f % COLS;
       v_r[m] = jj >= dv && jj < C ? 1.f : 0.f;
       if (tt < nc && jj < dv) v_r[m] = v[((size_t)start + c0 + tt) * v_stride + (size_t)h * dv + jj];
     }
@@ -545,63 +610,95 @@ decay_scan_kernel(float* __restrict__ out, int out_stride, const float* __restri
     for (int m = 0; m < NV4; ++m) {
       const int f = tid + m * kScanThreads;
       reinterpret_cast<float4*>(&k_s[0][0])[f] = k_r[m];
-      reinterpret_cast<float4*>(&q_s[0][0])[f] = q_r[m];
+      if (MODE != 1) reinterpret_cast<float4*>(&q_s[0][0])[f] = q_r[m];
     }
 #pragma unroll
     for (int m = 0; m < NV; ++m) (&v_s[0][0])[tid + m * kScanThreads] = v_r[m];
     if (tid < CH) { a_s[tid] = a_r; b_s[tid] = b_r; }
     __syncthreads();
     if (c0 + CH < n) fetch(c0 + CH);
-    auto token = [&](int tt) {                   // S <- a S + b v k, returns this lane's part of S^T q
-      const float aa = a_s[tt], bv = b_s[tt] * v_s[tt][col];
-      float acc[G4];
+    auto token = [&](int tt, float* sums) {      // S <- a S + b v k; sums: this lane's parts of S^T q
+      const float aa = a_s[tt];
+      float bv[CPL];
+      float acc[CPL][G4];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) bv[c] = b_s[tt] * v_s[tt][col + c * kScanCols];
 #pragma unroll
       for (int g = 0; g < G4; ++g) {
         const float4 kk = *reinterpret_cast<const float4*>(&k_s[tt][32 * g + 4 * lane]);
-        const float4 qq = *reinterpret_cast<const float4*>(&q_s[tt][32 * g + 4 * lane]);
-        S[g].x = fmaf(aa, S[g].x, bv * kk.x);
-        S[g].y = fmaf(aa, S[g].y, bv * kk.y);
-        S[g].z = fmaf(aa, S[g].z, bv * kk.z);
-        S[g].w = fmaf(aa, S[g].w, bv * kk.w);
-        acc[g] = fmaf(S[g].w, qq.w, fmaf(S[g].z, qq.z, fmaf(S[g].y, qq.y, S[g].x * qq.x)));
-      }
-      float sum = acc[0];
+        float4 qq;
+        if (MODE != 1) qq = *reinterpret_cast<const float4*>(&q_s[tt][32 * g + 4 * lane]);
 #pragma unroll
-      for (int g = 1; g < G4; ++g) sum += acc[g];
-      return sum;
+        for (int c = 0; c < CPL; ++c) {
+          float4& s4 = S[c][g];
+          s4.x = fmaf(aa, s4.x, bv[c] * kk.x);
+          s4.y = fmaf(aa, s4.y, bv[c] * kk.y);
+          s4.z = fmaf(aa, s4.z, bv[c] * kk.z);
+          s4.w = fmaf(aa, s4.w, bv[c] * kk.w);
+          if (MODE != 1) acc[c][g] = fmaf(s4.w, qq.w, fmaf(s4.z, qq.z, fmaf(s4.y, qq.y, s4.x * qq.x)));
+        }
+      }
+      if (MODE == 1) { prod *= aa; return; }
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        sums[c] = acc[c][0];
+#pragma unroll
+        for (int g = 1; g < G4; ++g) sums[c] += acc[c][g];
+      }
     };
     int tt = 0;
+    if (MODE == 1) {
+#pragma unroll 4
+      for (; tt < nc; ++tt) token(tt, nullptr);
+      continue;
+    }
     // eight tokens at a time: their partial sums are exchanged so that lane l ends with token l's total
     // (7 shuffles in 3 levels for 8 tokens instead of 24 in 24)
     for (; tt + 8 <= nc; tt += 8) {
-      float p[8];
+      float p8[8][CPL];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) p[u] = token(tt + u);
+      for (int u = 0; u < 8; ++u) token(tt + u, p8[u]);
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const float send = (lane & 4) ? p[u] : p[u + 4], keep = (lane & 4) ? p[u + 4] : p[u];
-        p[u] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+      for (int c = 0; c < CPL; ++c) {
+        float p[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) p[u] = p8[u][c];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const float send = (lane & 4) ? p[u] : p[u + 4], keep = (lane & 4) ? p[u + 4] : p[u];
+          p[u] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const float send = (lane & 2) ? p[u] : p[u + 2], keep = (lane & 2) ? p[u + 2] : p[u];
+          p[u] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
+        }
+        const float send = (lane & 1) ? p[0] : p[1], keep = (lane & 1) ? p[1] : p[0];
+        const float total = keep + __shfl_xor_sync(0xffffffffu, send, 1);
+        if (live[c]) out[(size_t)(start + c0 + tt + lane) * out_stride + (size_t)h * C + j[c]] = total;
       }
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const float send = (lane & 2) ? p[u] : p[u + 2], keep = (lane & 2) ? p[u + 2] : p[u];
-        p[u] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
-      }
-      const float send = (lane & 1) ? p[0] : p[1], keep = (lane & 1) ? p[1] : p[0];
-      const float total = keep + __shfl_xor_sync(0xffffffffu, send, 1);
-      if (live) out[(size_t)(start + c0 + tt + lane) * out_stride + (size_t)h * C + j] = total;
     }
     for (; tt < nc; ++tt) {
-      float sum = token(tt);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 4);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-      if (lane == 0 && live) out[(size_t)(start + c0 + tt) * out_stride + (size_t)h * C + j] = sum;
+      float sums[CPL];
+      token(tt, sums);
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        float sum = sums[c];
+        sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+        if (lane == 0 && live[c]) out[(size_t)(start + c0 + tt) * out_stride + (size_t)h * C + j[c]] = sum;
+      }
     }
   }
-  if (write_state && live) {
+  if (MODE == 1 && tid == 0 && blockIdx.z == 0) seg.prods[((size_t)seq * seg.count + part) * heads + h] = prod;
+  if (MODE == 1 || write_state) {
+    float* to = MODE == 1 ? carry_at(part + 1) : sp;
 #pragma unroll
-    for (int g = 0; g < G4; ++g) *reinterpret_cast<float4*>(sp + 32 * g + 4 * lane) = S[g];
+    for (int c = 0; c < CPL; ++c)
+#pragma unroll
+      for (int g = 0; g < G4; ++g)
+        if (live[c]) store(to, c, g, S[c][g]);
   }
 }
 
@@ -820,21 +917,34 @@ EK_EXPORT int ek_decay_scan(float* out, int out_stride, const float* q, int q_st
                             const float* v, int v_stride, const float* a, const float* b, float* state,
                             long long slot_stride, const int* cu_seqlens, const int* positions,
                             const int* token_slot, int n_seqs, int heads, int kv_heads, int dk, int dv,
-                            int ones_col, int write_state, int ab_stride, cudaStream_t stream) {
+                            int ones_col, int write_state, int ab_stride, float* carry, float* prods,
+                            int segments, int seg_len, int wide, cudaStream_t stream) {
   using namespace ek;
   if (n_seqs <= 0) return 0;
+  if (segments > 1 && (!carry || !prods || seg_len <= 0 || ((uintptr_t)carry & 15))) return EK_ERR_ARG;
   if (ab_stride != 0 && ab_stride != heads) return EK_ERR_ARG;
   const int rows = ek_decay_scan_rows(dk);
   if (!rows || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dv <= 0 || heads > 65535 || slot_stride % 4 ||
       ((uintptr_t)state & 15))
     return EK_ERR_ARG;
   const int C = dv + (ones_col ? 1 : 0);
-  dim3 grid(n_seqs, heads, (C + kScanCols - 1) / kScanCols);
-  auto kernel = rows == 32 ? decay_scan_kernel<4> : rows == 64 ? decay_scan_kernel<8>
-              : rows == 128 ? decay_scan_kernel<16> : decay_scan_kernel<32>;
-  return (int)launch_pdl(kernel, grid, dim3(kScanThreads), 0, stream, out, out_stride, q, q_stride, k, k_stride, v,
-                         v_stride, a, b, state, (size_t)slot_stride, cu_seqlens, positions, token_slot, heads,
-                         kv_heads, dk, dv, ones_col ? 1 : 0, write_state, ab_stride);
+  const bool cut = segments > 1;
+  const int cols = kScanCols * (wide ? 2 : 1);
+  dim3 grid(n_seqs * (cut ? segments : 1), heads, (C + cols - 1) / cols);
+  const ScanSegments seg{carry, prods, segments, seg_len};
+#define EK_SCAN_ROWS(MODE_, CPL_)                                                                               \
+  (rows == 32 ? decay_scan_kernel<4, MODE_, CPL_> : rows == 64 ? decay_scan_kernel<8, MODE_, CPL_>              \
+   : rows == 128 ? decay_scan_kernel<16, MODE_, CPL_> : decay_scan_kernel<32, MODE_, CPL_>)
+#define EK_SCAN(MODE_)                                                                                          \
+  (int)launch_pdl(wide ? EK_SCAN_ROWS(MODE_, 2) : EK_SCAN_ROWS(MODE_, 1), grid, dim3(kScanThreads), 0, stream,  \
+                  out, out_stride, q, q_stride, k, k_stride, v, v_stride, a, b, state, (size_t)slot_stride,     \
+                  cu_seqlens, positions, token_slot, heads, kv_heads, dk, dv, ones_col ? 1 : 0, write_state,    \
+                  ab_stride, seg)
+  if (!cut) return EK_SCAN(0);
+  const int rc = EK_SCAN(1);
+  return rc ? rc : EK_SCAN(2);
+#undef EK_SCAN
+#undef EK_SCAN_ROWS
 }
 
 // y[t, c] = rms-normed over all `inner` channels o * w[c] * sigmoid(proj[t, col_g + c]).  A block a token.

@@ -611,23 +611,39 @@ qk_whole_norm_rope_kv_kernel(T* rows, int row_stride, const float* __restrict__ 
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int D = cache.head_dim, n_kv = cache.heads, half = rot_dim >> 1;
   const int n_norm = write_kv ? n_q + n_kv : n_q, n_heads = write_kv ? n_q + 2 * n_kv : n_q;
-  const int pos = positions[t];
-  if (pos < 0) return;
   T* row = rows + (size_t)t * row_stride;
-  int page = 0;
-  if (write_kv) page = cache.block_table[(size_t)token_slot[t] * cache.table_stride + pos / EK_PAGE];
   const int per_head = vec ? D >> 2 : 1, head_step = (int)blockDim.x / per_head;
   const int head0 = tid / per_head, j = (tid % per_head) * 4;
   const bool mine = vec && head0 < head_step;
+  // the first heads are asked for before the position is known, the angles before the norms are
+  float4 v[kWholePasses];
+  auto load_heads = [&](int base) {
+#pragma unroll
+    for (int p = 0; p < kWholePasses; ++p) {
+      const int head = base + p * head_step;
+      if (head < n_heads) v[p] = Vec4<T>::load(row + (size_t)head * D + j);
+    }
+  };
+  if (mine) load_heads(head0);
+  const int pos = positions[t];
+  if (pos < 0) return;
+  int page = 0;
+  if (write_kv) page = cache.block_table[(size_t)token_slot[t] * cache.table_stride + pos / EK_PAGE];
+  const float* cs = cos_tab + (size_t)pos * half;
+  const float* sn = sin_tab + (size_t)pos * half;
+  float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
+  int partner = j;
+  if (mine && j < rot_dim) {
+    const int a = j < half ? j : j - half;
+    c = *reinterpret_cast<const float4*>(cs + a);
+    s = *reinterpret_cast<const float4*>(sn + a);
+    if (j < half) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+    partner = j < half ? j + half : j - half;
+  }
   float sq = 0.f, sk = 0.f;
   if (mine) {
     for (int base = head0; base < n_heads; base += head_step * kWholePasses) {
-      float4 v[kWholePasses];
-#pragma unroll
-      for (int p = 0; p < kWholePasses; ++p) {
-        const int head = base + p * head_step;
-        if (head < n_heads) v[p] = Vec4<T>::load(row + (size_t)head * D + j);
-      }
+      if (base > head0) load_heads(base);
 #pragma unroll
       for (int p = 0; p < kWholePasses; ++p) {
         const int head = base + p * head_step;
@@ -666,18 +682,7 @@ qk_whole_norm_rope_kv_kernel(T* rows, int row_stride, const float* __restrict__ 
   sq = sk = 0.f;
   for (int w = 0; w < n_warps; ++w) { sq += part_q[w]; sk += part_k[w]; }
   const float rq = rsqrtf(sq / (float)(n_q * norm_dim) + eps), rk = rsqrtf(sk / (float)(n_kv * norm_dim) + eps);
-  const float* cs = cos_tab + (size_t)pos * half;
-  const float* sn = sin_tab + (size_t)pos * half;
   if (mine) {
-    float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
-    int partner = j;
-    if (j < rot_dim) {
-      const int a = j < half ? j : j - half;
-      c = *reinterpret_cast<const float4*>(cs + a);
-      s = *reinterpret_cast<const float4*>(sn + a);
-      if (j < half) s = make_float4(-s.x, -s.y, -s.z, -s.w);
-      partner = j < half ? j + half : j - half;
-    }
     for (int head = head0; head < n_norm; head += head_step) {
       const float r = head < n_q ? rq : rk;
       const float4 x = *reinterpret_cast<const float4*>(vals + (size_t)head * D + j);

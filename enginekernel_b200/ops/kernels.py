@@ -1650,7 +1650,7 @@ _xgate_scan = Function("recurrent", "ek_xgate_scan",
                         c_int, c_int, c_int, _P])
 _decay_scan = Function("recurrent", "ek_decay_scan",
                        [_P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_longlong, _P, _P, _P,
-                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P])
+                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, c_int, c_int, _P])
 _ssm_out = _per_dtype("recurrent", "ek_ssm_out",
                       [_P, _P, _P, c_int, _P, c_int, c_int, _P, _P, c_float, _P, c_int, c_int, c_int, c_int, _P])
 _xlstm_out = _per_dtype("recurrent", "ek_xlstm_out",
@@ -1787,13 +1787,38 @@ def xgate_scan(a, b, m_run, proj, col_i, col_f, bias_i, bias_f, cap, state, m_of
                 _ptr(token_slot), n_seqs, heads, 1 if write_state else 0, _stream())
 
 
+SCAN_COLUMNS = 16           # columns of S a block of the decay scan takes, one a lane; twice as many with two
+SCAN_WIDE_TOKENS = 64       # sequences of at least this many tokens take two columns a lane
+SCAN_BLOCKS_PER_SM = 6      # what a cut of long prompts into segments aims at
+SCAN_MIN_SEGMENT = 128      # tokens
+SCAN_MIN_SEGMENTS = 4       # (the walk of the states costs two thirds of a walk: two or three segments gain nothing)
+
+
+def decay_scan_wide(columns, max_new) -> bool:
+    """Whether a lane of :func:`decay_scan` takes two columns (long walks of enough columns)."""
+    return max_new >= SCAN_WIDE_TOKENS and columns > SCAN_COLUMNS
+
+
+def decay_scan_segments(n_seqs, heads, columns, max_new, device=None):
+    """(segments of the longest sequence, tokens a segment) that :func:`decay_scan` cuts a step's sequences into; one
+    segment where the sequences, heads and columns fill the machine, or the sequences are short."""
+    tile = SCAN_COLUMNS * (2 if decay_scan_wide(columns, max_new) else 1)
+    blocks = n_seqs * heads * -(-columns // tile)
+    want = min(SCAN_BLOCKS_PER_SM * sm_count(device) // blocks, max_new // SCAN_MIN_SEGMENT)
+    if want < SCAN_MIN_SEGMENTS:
+        return 1, max_new
+    length = -(-(-(-max_new // want)) // 64) * 64
+    return -(-max_new // length), length
+
+
 def decay_scan(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot, n_seqs, heads, kv_heads, dim, vdim,
-               ones_column=False, write_state=True, n_tokens=0):
+               ones_column=False, write_state=True, n_tokens=0, max_new=0, workspace=None, segments=None):
     """S_t = a_t S_(t-1) + b_t k_t v_t^T, out_t = S_t^T q_t per head over every sequence's tokens, S
     ([heads, columns, rows] at the start of a slot's state, 32-bit) read and written back.  ``q``, ``k``
     [T, >= kv_heads * dim] (head h reads key head h // (heads / kv_heads)), ``v`` [T, >= heads * vdim],
     ``a``, ``b`` [T, heads], or [heads] where they are the same for every token.  ``ones_column``: one more column whose v is 1 (it carries a n + b k and
-    gives n . q); out is [T, heads * columns]."""
+    gives n . q); out is [T, heads * columns].  With ``workspace`` and ``max_new`` (tokens of the longest sequence) long
+    sequences are cut into segments that run side by side (:func:`decay_scan_segments`, or ``segments`` as given)."""
     _need_cuda(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot)
     _need_f32("decay_scan", out, q, k, v, a, b, state)
     cols = vdim + (1 if ones_column else 0)
@@ -1805,10 +1830,20 @@ def decay_scan(out, q, k, v, a, b, state, cu_seqlens, positions, token_slot, n_s
         lib.annotate(bytes=4 * (n_tokens * (2 * kv_heads * dim + 2 * heads * vdim + 2 * heads)
                                 + 2 * n_seqs * heads * cols * decay_scan_rows(dim)),
                      flops=4 * n_tokens * heads * dim * cols)
+    parts, length, carry, prods = 1, 0, None, None
+    if workspace is not None and max_new > 1:
+        parts, length = segments or decay_scan_segments(n_seqs, heads, cols, max_new, out.device)
+        _need(length >= 1 and parts * length >= max_new, "decay_scan: the segments cover the longest sequence")
+        if parts > 1:
+            carry = workspace.get("scan_carry", (n_seqs, parts, heads * cols * decay_scan_rows(dim)), torch.float32)
+            prods = workspace.get("scan_prods", (n_seqs, parts, heads), torch.float32)
     _decay_scan(_ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
                 _ptr(a), _ptr(b), _ptr(state), state.stride(0), _ptr(cu_seqlens), _ptr(positions), _ptr(token_slot),
                 n_seqs, heads, kv_heads, dim, vdim, 1 if ones_column else 0, 1 if write_state else 0,
-                heads if a.dim() > 1 else 0, _stream())
+                heads if a.dim() > 1 else 0, _ptr(carry), _ptr(prods), parts, length,
+                1 if decay_scan_wide(cols, max_new) else 0, _stream())
+    if parts > 1:
+        count_extra_launches()
 
 
 def ssm_out(y, o, x, proj, col_z, d_skip, w, eps, positions, n_tokens, inner, vdim, parts):
@@ -1889,7 +1924,7 @@ def xlstm_out(y, o, m_run, proj, col_g, w, eps, q_scale, positions, n_tokens, he
 
 
 # ------------------------------------------------------------------ routed experts
-_moe_route = Function("moe", "ek_moe_route", [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P])
+_moe_route = Function("moe", "ek_moe_route", [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P])
 _moe_plan = Function("moe", "ek_moe_plan", [_P, _P, _P, _P, c_int, c_int, _P])
 _moe_up = _per_dtype("moe", "ek_moe_expert_up",
                      [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P])
@@ -1925,9 +1960,9 @@ def moe_route(sel_expert, sel_weight, logits, n_tokens, n_groups, keep, top, sca
                                  and correction.numel() == logits.shape[-1]),
           "moe_route: a 32-bit correction per expert goes with the weights 'softmax'")
     _need(weights in ROUTE_WEIGHTS, f"moe_route: no weights {weights!r}")
-    _need(logits.dtype == torch.float32 and logits.is_contiguous() and sel_expert.dtype == torch.int32
+    _need(logits.dtype == torch.float32 and logits.stride(-1) == 1 and sel_expert.dtype == torch.int32
           and sel_weight.dtype == torch.float32, "moe_route: 32-bit logits and weights, int32 choices")
-    _moe_route(_ptr(sel_expert), _ptr(sel_weight), _ptr(logits), n_tokens, logits.shape[-1], n_groups, keep,
+    _moe_route(_ptr(sel_expert), _ptr(sel_weight), _ptr(logits), logits.stride(0), n_tokens, logits.shape[-1], n_groups, keep,
                top, float(scale), ROUTE_WEIGHTS[weights], _ptr(correction), _stream())
 
 

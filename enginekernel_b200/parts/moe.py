@@ -102,7 +102,8 @@ class RoutedExperts(FeedForward):
         w = self.spec.weights
         if self.shared is not None:
             self.shared.load(tensors)
-        self.w_router = tensors[w["router"]].to(self.dtype).contiguous()
+        router = tensors[w["router"]]           # (zero rows up to a multiple of 16: the library is slow on a ragged few)
+        self.w_router = torch.cat([router, router.new_zeros((-self.routed % 16, self.hidden))], 0).to(self.dtype).contiguous()
         if self.corrected:
             self.correction = tensors[w["correction"]].to(torch.float32).contiguous()
         ups = [tensors[w[f"up_{e}"]] for e in range(self.experts)]
@@ -125,7 +126,7 @@ class RoutedExperts(FeedForward):
         logits = linear(x, self.w_router, ctx, "router_logits", n_rows=t, out_dtype=torch.float32, wide_f32="library")
         chosen = ws.get("moe_chosen", (t, top), torch.int32)
         weight = ws.get("moe_weight", (t, top), torch.float32)
-        kernels.moe_route(chosen, weight, logits, t, self.groups, self.keep, top, self.scale,
+        kernels.moe_route(chosen, weight, logits[:, :self.routed], t, self.groups, self.keep, top, self.scale,
                           weights=self.weights, correction=self.correction)
         sorted_pair = ws.get("moe_sorted", (pairs,), torch.int32)
         tiles = ws.get("moe_tiles", (kernels.moe_max_tiles(pairs, self.experts), 3), torch.int32)

@@ -121,7 +121,7 @@ class StateSpace(Mixer):
         o = ws.get("scan_o", (t, inner), f32)
         kernels.decay_scan(o, xbc[:, inner + g * n:], xbc[:, inner:inner + g * n], xbc, a, b, state,
                            ctx.cu_seqlens, ctx.positions, ctx.token_slot, ctx.n_seqs, nh, g, n, e,
-                           write_state=writes_cache, n_tokens=t)
+                           write_state=writes_cache, n_tokens=t, max_new=ctx.max_new, workspace=ws)
         y = ws.get("attn_out", (t, inner), self.dtype)
         kernels.ssm_out(y, o, xbc, proj, 0, self.d_skip, self.norm_w, self.eps, ctx.positions, t, inner, e,
                         self.norm_groups)
@@ -180,7 +180,7 @@ class MatrixMemory(Mixer):
         o = ws.get("scan_o", (t, nh * (e + 1)), f32)
         kernels.decay_scan(o, proj, proj[:, col_k:], proj[:, col_v:], a, b, state, ctx.cu_seqlens, ctx.positions,
                            ctx.token_slot, ctx.n_seqs, nh, nh, d, e, ones_column=True, write_state=writes_cache,
-                           n_tokens=t)
+                           n_tokens=t, max_new=ctx.max_new, workspace=ws)
         y = ws.get("attn_out", (t, nh * e), self.dtype)
         kernels.xlstm_out(y, o, m_run, proj, col_g, self.norm_w, self.eps, d ** -0.5, ctx.positions, t, nh, e)
         return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
@@ -238,7 +238,8 @@ class FixedDecayMemory(Mixer):
         kernels.bias_act(qkv, proj, None, "silu", n_rows=t)
         o = ws.get("scan_o", (t, nh * e), f32)
         kernels.decay_scan(o, qkv, qkv[:, nh * d:], qkv[:, 2 * nh * d:], self.a, self.b, entry.state, ctx.cu_seqlens,
-                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache, n_tokens=t)
+                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache,
+                           n_tokens=t, max_new=ctx.max_new, workspace=ws)
         y = ws.get("attn_out", (t, nh * e), self.dtype)
         kernels.norm_gate_out(y, o, proj, width, self.norm_w, self.eps, ctx.positions, t)
         return linear(y, self.w_o, ctx, "attn_proj", n_rows=t)
@@ -307,7 +308,8 @@ class Retention(Mixer):
             kernels.rotate_heads(proj, 0, 2 * nh, d, pos.rotary_dim, pos.cos, pos.sin, ctx.positions, t)
         o = ws.get("scan_o", (t, nh * e), f32)
         kernels.decay_scan(o, proj, proj[:, nh * d:], proj[:, 2 * nh * d:], self.a, self.b, entry.state, ctx.cu_seqlens,
-                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache, n_tokens=t)
+                           ctx.positions, ctx.token_slot, ctx.n_seqs, nh, nh, d, e, write_state=writes_cache,
+                           n_tokens=t, max_new=ctx.max_new, workspace=ws)
         y = ws.get("attn_out", (t, nh * e), self.dtype)
         kernels.head_norm_gate_out(y, o, proj, nh * (2 * d + e), None, self.eps, ctx.positions, t, nh, e,
                                    gate_activation="silu")

@@ -12,6 +12,7 @@ router's choice to be far from trivial.
 
 from __future__ import annotations
 
+import copy
 import json
 import math
 import os
@@ -66,7 +67,7 @@ def config(width, vocab, layers, eps=1e-5, logit_scale=0.7, logit_softcap=4.0):
     made = []
     for entry in layers:
         if isinstance(entry, int):
-            src = {k: v for k, v in made[entry].items() if k != "weights_of"}
+            src = {k: v for k, v in copy.deepcopy(made[entry]).items() if k != "weights_of"}
             made.append(dict(src, weights_of=entry))
         else:
             made.append(dict(entry[0], mlp=entry[1]))
@@ -95,7 +96,7 @@ ODD = config(100, 89, [
     (latent(2, 12, 6, 28, 10, 1), moe(3, 1, 3, 12, 20)),
     (attention(3, 3, 20, 20, rotation(10, 1e6, (2.0, 100, 4.0, 1.0)), None), None),
     (latent(5, 20, 10, 12, 70, 33), None),
-    1], eps=1e-4, logit_scale=2.5, logit_softcap=2.0)
+    1], eps=1e-4, logit_scale=1.3, logit_softcap=3.0)
 # heads of 64 and 128: the kernels on tcgen05 and those fed by TMA; more shared and identity experts
 WIDE = config(256, 301, [
     (attention(8, 2, 128, 128, rotation(64, 1e5, (4.0, 512, 32.0, 1.0)), 130), moe(7, 9, 3, 64, 96)),
